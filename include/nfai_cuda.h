@@ -39,7 +39,7 @@ enum {
   NFAI_ERR_TIMEOUT = 7       /* a bounded device-side wait gave up */
 };
 
-enum { NFAI_F32 = 0, NFAI_F16 = 1 };
+enum { NFAI_F32 = 0, NFAI_F16 = 1, NFAI_BF16 = 2 /* weights of layer-plan models; any tensor upload */ };
 
 /* Model geometry. Mirrors what the reference reads from GGUF metadata
  * (NFAI.Models.Llama3/LlamaModel.cs:23-39) plus ModelOptions.KVCacheSize (NFAI.Models/ModelOptions.cs:3-8). */
@@ -155,6 +155,26 @@ int nfai_gguf_probe(const char* path, uint32_t kv_cache_size, nfai_hparams* out,
 /* The model's geometry as it was created (filled by nfai_model_load_gguf from the file). */
 int nfai_model_get_hparams(const nfai_model* m, nfai_hparams* out);
 
+/* ---- models described by a configuration (layer plans) -------------------------------------------------------
+ * A model folder holds config.json, whose "architecture" names the design and whose "layers" list every layer's mixer
+ * (its kind and sizes) and feed-forward, and model.safetensors. Known architectures: "Tometar" (hyper-connected
+ * residual streams, latent attention with a sliding window, Mamba-2 layers, relu-gated feed-forwards). The handle is an
+ * nfai_model like any other: prefill, decode, greedy and sampled loops, snapshots and taps work on it. Differences:
+ * nfai_set_position only goes to 0 or the current position (recurrent state), one GPU, the cache has the weights' type,
+ * nfai_read_kv returns the latent (kv_rank floats) as k and the shared rotated key part (rot_dim floats) as v of a latent
+ * attention layer, nfai_read_hidden the sum of the streams. weight_dtype: NFAI_BF16 (served precision) or NFAI_F32 (true
+ * 32-bit everywhere). No counterpart in the reference, whose one model family is Llama
+ * (NFAI.Models.Llama3/LlamaModelFactory.cs:36-44). */
+int nfai_model_create_from_config(nfai_ctx* ctx, const char* config_json, size_t len, uint32_t kv_cache_size,
+                                  int weight_dtype, nfai_model** out);
+/* create_from_config + upload of every tensor the plan needs from <dir>/model.safetensors (memory-mapped, offsets and
+ * sizes checked against the file) + nfai_model_finalize. */
+int nfai_model_load_dir(nfai_ctx* ctx, const char* dir, uint32_t kv_cache_size, int weight_dtype, nfai_model** out);
+/* Check a configuration without a device: geometry into `out` (may be null), and one line "name dim0 dim1 ..." per tensor
+ * the model needs (outermost dimension first) into tensors_out (may be null; *n_out = length without the final zero). */
+int nfai_config_probe(const char* config_json, size_t len, nfai_hparams* out, char* tensors_out, size_t cap, size_t* n_out,
+                      char* err_out, size_t err_bytes);
+
 /* replaces: LlamaModel.Dispose (LlamaModel.cs:70-74, which throws NotImplementedException). */
 int nfai_model_destroy(nfai_model* m);
 
@@ -165,6 +185,11 @@ int nfai_model_destroy(nfai_model* m);
  * The result equals feeding the tokens one by one through nfai_decode.
  * replaces: the prompt loop of LlamaModel.RunAsync (LlamaModel.cs:103-126). */
 int nfai_prefill(nfai_model* m, const uint32_t* tokens, int n, float* logits_last, uint32_t* argmax_last);
+
+/* n tokens at positions pos .. pos+n-1 with the logits of chosen places among them: `want` holds n_want ascending indices
+ * below n, `logits` receives n_want rows of V floats (n_want = 0: none). Equals feeding the tokens one by one through
+ * nfai_decode; the place of the cut between calls makes no difference beyond rounding. No counterpart in the reference. */
+int nfai_forward(nfai_model* m, const uint32_t* tokens, int n, const uint32_t* want, int n_want, float* logits);
 
 /* One token at the current position: embed -> L x block -> output norm -> LM head. `logits` (V floats) and
  * `argmax` are optional host outputs. Advances the position by one.
@@ -229,6 +254,8 @@ int nfai_read_hidden(nfai_model* m, uint32_t layer, float* out);
  * events; launch i uses layer (i mod L)'s weights so that consecutive launches read different HBM.
  * which: 0 = FFN gate/up GEMV (+RMSNorm, +SiLU*up), 1 = FFN down GEMV (+residual), 2 = QKV GEMV (+RMSNorm,+RoPE),
  *        3 = O-projection GEMV (+residual), 4 = LM-head GEMV (+RMSNorm, +arg-max partials), 5 = attention.
+ *        Layer-plan models: 0 and 1 feed-forward, 2 input projection, 3 output projection and 5 attention of latent
+ *        attention layers, 4 LM head, 6 input projection, 7 step and 8 output projection of state space layers.
  * avg_ms receives the mean duration of one launch; bytes_per_launch the algorithmic bytes it must move. */
 int nfai_profile_kernel(nfai_model* m, int which, int iters, float* avg_ms, uint64_t* bytes_per_launch);
 

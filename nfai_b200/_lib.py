@@ -12,7 +12,7 @@ LIB_PATH = os.path.join(HERE, "lib", "libnfai_cuda.so")
 
 OK = 0
 ERR_ARG, ERR_STATE, ERR_OOM, ERR_CUDA, ERR_NCCL, ERR_CONTEXT_FULL, ERR_TIMEOUT = 1, 2, 3, 4, 5, 6, 7
-F32, F16 = 0, 1
+F32, F16, BF16 = 0, 1, 2
 
 ERROR_NAMES = {
     ERR_ARG: "NFAI_ERR_ARG", ERR_STATE: "NFAI_ERR_STATE", ERR_OOM: "NFAI_ERR_OOM", ERR_CUDA: "NFAI_ERR_CUDA",
@@ -61,9 +61,13 @@ SIGNATURES = {
     "nfai_model_finalize": (_i, [_vp]),
     "nfai_model_load_gguf": (_i, [_vp, C.c_char_p, _u32, _i, _pp]),
     "nfai_gguf_probe": (_i, [C.c_char_p, _u32, C.POINTER(HParams), C.c_char_p, _sz]),
+    "nfai_config_probe": (_i, [C.c_char_p, _sz, C.POINTER(HParams), C.c_char_p, _sz, C.POINTER(_sz), C.c_char_p, _sz]),
+    "nfai_model_create_from_config": (_i, [_vp, C.c_char_p, _sz, _u32, _i, _pp]),
+    "nfai_model_load_dir": (_i, [_vp, C.c_char_p, _u32, _i, _pp]),
     "nfai_model_get_hparams": (_i, [_vp, C.POINTER(HParams)]),
     "nfai_model_destroy": (_i, [_vp]),
     "nfai_prefill": (_i, [_vp, C.POINTER(_u32), _i, C.POINTER(_f), C.POINTER(_u32)]),
+    "nfai_forward": (_i, [_vp, C.POINTER(_u32), _i, C.POINTER(_u32), _i, C.POINTER(_f)]),
     "nfai_decode": (_i, [_vp, _u32, C.POINTER(_f), C.POINTER(_u32)]),
     "nfai_decode_greedy": (_i, [_vp, _u32, _i, C.POINTER(_u32), C.POINTER(_f)]),
     "nfai_decode_sampled": (_i, [_vp, _u32, _i, _f, _f, _i, _vp, _vp, C.POINTER(_f)]),

@@ -3,12 +3,14 @@
 The reference's toolchain (.NET) is not available where this package is developed, so the same call sequence a
 C# NFAI.Cuda project makes through P/Invoke is driven from here through ctypes, with the reference's names:
 ModelOptions, LlamaModelFactory.TryCreate, LlamaModel (NFAI.Models/ModelOptions.cs, NFAI.Models.Llama3/
-LlamaModelFactory.cs, LlamaModel.cs). Token ids go in and come out (the tokenizer is untouched CPU string code).
+LlamaModelFactory.cs, LlamaModel.cs). Models of other designs (PlannedModel: a folder with config.json and
+model.safetensors) share the same base class, step functions and samplers. Token ids go in and come out (the tokenizer is untouched CPU string code).
 Every compute step runs in libnfai_cuda.so; nothing here falls back to the CPU.
 """
 from __future__ import annotations
 
 import ctypes as C
+import json
 import os
 from dataclasses import dataclass
 from typing import Dict, Iterable, List, Optional, Sequence, Tuple
@@ -16,7 +18,7 @@ from typing import Dict, Iterable, List, Optional, Sequence, Tuple
 import numpy as np
 
 from . import _lib
-from ._lib import F16, F32, HParams, NfaiError, check
+from ._lib import BF16, F16, F32, HParams, NfaiError, check
 from .gguf_io import ComputeCollection
 
 
@@ -28,6 +30,7 @@ class ModelOptions:
     KVCacheDType: str = "auto"   # "f32" (the reference's cache type), "f16", or "auto" = the weights' type
     Device: int = 0
     WeightDType: str = "auto"    # "auto" = as stored in the file
+    ModelPath: str = ""          # a folder with config.json and model.safetensors instead of a GGUF file
 
 
 class CudaContext:
@@ -73,10 +76,142 @@ class CudaContext:
 
 
 def _dtype_code(name: str) -> int:
-    return {"f32": F32, "f16": F16}[name]
+    return {"f32": F32, "f16": F16, "bf16": BF16}[name]
 
 
-class LlamaModel:
+def _dtype_name(code: int) -> str:
+    return {F32: "f32", F16: "f16", BF16: "bf16"}[code]
+
+
+class CausalModel:
+    """What every model has over its nfai_model handle: the step functions, samplers, snapshots, taps and timers."""
+
+    ctx: CudaContext
+    handle: Optional[C.c_void_p]
+    eos_token = None
+
+    # -- the hot path -------------------------------------------------------------------------------------------
+    def _fp(self, a: Optional[np.ndarray]):
+        return a.ctypes.data_as(C.POINTER(C.c_float)) if a is not None else None
+
+    def prefill(self, tokens: Iterable[int], want_logits: bool = True) -> Tuple[Optional[np.ndarray], int]:
+        toks = np.ascontiguousarray(np.fromiter((int(t) for t in tokens), dtype=np.uint32))
+        logits = np.empty(self.V, np.float32) if want_logits else None
+        am = C.c_uint32()
+        check(self._lib.nfai_prefill(self.handle, toks.ctypes.data_as(C.POINTER(C.c_uint32)), toks.size,
+                                     self._fp(logits), C.byref(am)), self.ctx.handle)
+        return logits, am.value
+
+    def forward(self, tokens: Iterable[int], want: Sequence[int] = ()) -> np.ndarray:
+        """Feed `tokens`; logits [len(want)][V] of the places `want` (ascending) among them."""
+        toks = np.ascontiguousarray(np.fromiter((int(t) for t in tokens), dtype=np.uint32))
+        places = np.ascontiguousarray(want, np.uint32)
+        logits = np.empty((places.size, self.V), np.float32)
+        u32p = C.POINTER(C.c_uint32)
+        check(self._lib.nfai_forward(self.handle, toks.ctypes.data_as(u32p), toks.size, places.ctypes.data_as(u32p),
+                                     places.size, self._fp(logits)), self.ctx.handle)
+        return logits
+
+    def decode(self, token: int, want_logits: bool = True) -> Tuple[Optional[np.ndarray], int]:
+        logits = np.empty(self.V, np.float32) if want_logits else None
+        am = C.c_uint32()
+        check(self._lib.nfai_decode(self.handle, int(token), self._fp(logits), C.byref(am)), self.ctx.handle)
+        return logits, am.value
+
+    def decode_greedy(self, first_token: int, n_steps: int) -> Tuple[np.ndarray, float]:
+        out = np.empty(n_steps, np.uint32)
+        ms = C.c_float()
+        check(self._lib.nfai_decode_greedy(self.handle, int(first_token), n_steps,
+                                           out.ctypes.data_as(C.POINTER(C.c_uint32)), C.byref(ms)), self.ctx.handle)
+        return out, ms.value
+
+    def decode_sampled(self, first_token: int, us: Sequence[float], temperature: float = 0.5, top_p: float = 0.95,
+                       top_k: int = 40) -> Tuple[np.ndarray, float]:
+        """len(us) steps with SamplingUtils.TopP after each, fed back on the device; returns (tokens, milliseconds)."""
+        u = np.ascontiguousarray(us, np.float32)
+        out = np.empty(len(u), np.uint32)
+        ms = C.c_float()
+        check(self._lib.nfai_decode_sampled(self.handle, int(first_token), len(u), temperature, top_p, top_k,
+                                            u.ctypes.data_as(C.c_void_p), out.ctypes.data_as(C.c_void_p), C.byref(ms)),
+              self.ctx.handle)
+        return out, ms.value
+
+    def snapshot(self) -> "KvSnapshot":
+        """Copy of the cache rows, logits and position at this point (device memory); restore() rewinds to it."""
+        h = C.c_void_p()
+        check(self._lib.nfai_kv_snapshot_create(self.handle, C.byref(h)), self.ctx.handle)
+        return KvSnapshot(self, h)
+
+    def sample_top_p(self, temperature: float = 0.5, top_p: float = 0.95, top_k: int = 40, u: float = 0.5) -> int:
+        """SamplingUtils.TopP on the device over the last step's logits; `u` is the uniform draw."""
+        tok = C.c_uint32()
+        check(self._lib.nfai_sample_top_p(self.handle, temperature, top_p, top_k, u, C.byref(tok)), self.ctx.handle)
+        return tok.value
+
+    def run_tokens(self, prompt: Iterable[int], max_new: int, stop_at_eos: bool = False) -> List[int]:
+        """LlamaModel.RunAsync with token ids in place of text and arg-max in place of TopP
+        (LlamaModel.cs:99-174): ingest the prompt, then feed each prediction back."""
+        _, tk = self.prefill(prompt, want_logits=False)
+        out = [tk]
+        while len(out) < max_new and not (stop_at_eos and tk == self.eos_token):
+            _, tk = self.decode(tk, want_logits=False)
+            out.append(tk)
+        return out
+
+    @property
+    def position(self) -> int:
+        p = C.c_uint32()
+        check(self._lib.nfai_position(self.handle, C.byref(p)), self.ctx.handle)
+        return p.value
+
+    def reset(self):
+        check(self._lib.nfai_reset(self.handle), self.ctx.handle)
+
+    def set_position(self, pos: int):
+        check(self._lib.nfai_set_position(self.handle, int(pos)), self.ctx.handle)
+
+    # -- taps ---------------------------------------------------------------------------------------------------
+    def read_hidden(self, layer: int) -> np.ndarray:
+        out = np.empty(self.H, np.float32)
+        check(self._lib.nfai_read_hidden(self.handle, layer, self._fp(out)), self.ctx.handle)
+        return out
+
+    # -- measurement --------------------------------------------------------------------------------------------
+    KERNELS = {"ffn_gate_up": 0, "ffn_down": 1, "qkv_rope": 2, "attn_out": 3, "lm_head": 4, "attention": 5}
+
+    def profile_kernel(self, which: str, iters: int) -> Tuple[float, int]:
+        ms = C.c_float()
+        nbytes = C.c_uint64()
+        check(self._lib.nfai_profile_kernel(self.handle, self.KERNELS[which], iters, C.byref(ms), C.byref(nbytes)),
+              self.ctx.handle)
+        return ms.value, nbytes.value
+
+    def tune(self, which: str, mode: int, rows_per_warp: int, depth: int, ctas_per_sm: int):
+        check(self._lib.nfai_model_tune(self.handle, self.KERNELS[which], mode, rows_per_warp, depth, ctas_per_sm),
+              self.ctx.handle)
+
+    def set_prefetch(self, lookahead_bytes: int, extra_bytes: int = 0, mode: int = 1):
+        check(self._lib.nfai_model_set_prefetch(self.handle, int(lookahead_bytes), int(extra_bytes), mode),
+              self.ctx.handle)
+
+    def step_launches(self) -> int:
+        n = C.c_int()
+        check(self._lib.nfai_step_launches(self.handle, C.byref(n)), self.ctx.handle)
+        return n.value
+
+    def Dispose(self):
+        if getattr(self, "handle", None):
+            self._lib.nfai_model_destroy(self.handle)
+            self.handle = None
+
+    def __del__(self):
+        try:
+            self.Dispose()
+        except Exception:
+            pass
+
+
+class LlamaModel(CausalModel):
     """IInferenceProvider for general.architecture == "llama" (NFAI.Models.Llama3/LlamaModel.cs:10-175).
 
     The constructor reads the same metadata keys as the reference (:23-39), finds the same tensors (:43,58 and
@@ -157,76 +292,6 @@ class LlamaModel:
             check(self._lib.nfai_model_tensor_chunk(self.handle, chunk, len(chunk)), self.ctx.handle)
         check(self._lib.nfai_model_tensor_end(self.handle), self.ctx.handle)
 
-    # -- the hot path -------------------------------------------------------------------------------------------
-    def _fp(self, a: Optional[np.ndarray]):
-        return a.ctypes.data_as(C.POINTER(C.c_float)) if a is not None else None
-
-    def prefill(self, tokens: Iterable[int], want_logits: bool = True) -> Tuple[Optional[np.ndarray], int]:
-        toks = np.ascontiguousarray(np.fromiter((int(t) for t in tokens), dtype=np.uint32))
-        logits = np.empty(self.V, np.float32) if want_logits else None
-        am = C.c_uint32()
-        check(self._lib.nfai_prefill(self.handle, toks.ctypes.data_as(C.POINTER(C.c_uint32)), toks.size,
-                                     self._fp(logits), C.byref(am)), self.ctx.handle)
-        return logits, am.value
-
-    def decode(self, token: int, want_logits: bool = True) -> Tuple[Optional[np.ndarray], int]:
-        logits = np.empty(self.V, np.float32) if want_logits else None
-        am = C.c_uint32()
-        check(self._lib.nfai_decode(self.handle, int(token), self._fp(logits), C.byref(am)), self.ctx.handle)
-        return logits, am.value
-
-    def decode_greedy(self, first_token: int, n_steps: int) -> Tuple[np.ndarray, float]:
-        out = np.empty(n_steps, np.uint32)
-        ms = C.c_float()
-        check(self._lib.nfai_decode_greedy(self.handle, int(first_token), n_steps,
-                                           out.ctypes.data_as(C.POINTER(C.c_uint32)), C.byref(ms)), self.ctx.handle)
-        return out, ms.value
-
-    def decode_sampled(self, first_token: int, us: Sequence[float], temperature: float = 0.5, top_p: float = 0.95,
-                       top_k: int = 40) -> Tuple[np.ndarray, float]:
-        """len(us) steps with SamplingUtils.TopP after each, fed back on the device; returns (tokens, milliseconds)."""
-        u = np.ascontiguousarray(us, np.float32)
-        out = np.empty(len(u), np.uint32)
-        ms = C.c_float()
-        check(self._lib.nfai_decode_sampled(self.handle, int(first_token), len(u), temperature, top_p, top_k,
-                                            u.ctypes.data_as(C.c_void_p), out.ctypes.data_as(C.c_void_p), C.byref(ms)),
-              self.ctx.handle)
-        return out, ms.value
-
-    def snapshot(self) -> "KvSnapshot":
-        """Copy of the cache rows, logits and position at this point (device memory); restore() rewinds to it."""
-        h = C.c_void_p()
-        check(self._lib.nfai_kv_snapshot_create(self.handle, C.byref(h)), self.ctx.handle)
-        return KvSnapshot(self, h)
-
-    def sample_top_p(self, temperature: float = 0.5, top_p: float = 0.95, top_k: int = 40, u: float = 0.5) -> int:
-        """SamplingUtils.TopP on the device over the last step's logits; `u` is the uniform draw."""
-        tok = C.c_uint32()
-        check(self._lib.nfai_sample_top_p(self.handle, temperature, top_p, top_k, u, C.byref(tok)), self.ctx.handle)
-        return tok.value
-
-    def run_tokens(self, prompt: Iterable[int], max_new: int, stop_at_eos: bool = False) -> List[int]:
-        """LlamaModel.RunAsync with token ids in place of text and arg-max in place of TopP
-        (LlamaModel.cs:99-174): ingest the prompt, then feed each prediction back."""
-        _, tk = self.prefill(prompt, want_logits=False)
-        out = [tk]
-        while len(out) < max_new and not (stop_at_eos and tk == self.eos_token):
-            _, tk = self.decode(tk, want_logits=False)
-            out.append(tk)
-        return out
-
-    @property
-    def position(self) -> int:
-        p = C.c_uint32()
-        check(self._lib.nfai_position(self.handle, C.byref(p)), self.ctx.handle)
-        return p.value
-
-    def reset(self):
-        check(self._lib.nfai_reset(self.handle), self.ctx.handle)
-
-    def set_position(self, pos: int):
-        check(self._lib.nfai_set_position(self.handle, int(pos)), self.ctx.handle)
-
     # -- taps ---------------------------------------------------------------------------------------------------
     def _kv_len(self) -> int:
         return self.hp.kvH * self.hp.d // self.ctx.world
@@ -250,57 +315,94 @@ class LlamaModel:
         check(self._lib.nfai_write_kv_range(self.handle, layer, pos0, k.shape[0], self._fp(k), self._fp(v)),
               self.ctx.handle)
 
-    def read_hidden(self, layer: int) -> np.ndarray:
-        out = np.empty(self.H, np.float32)
-        check(self._lib.nfai_read_hidden(self.handle, layer, self._fp(out)), self.ctx.handle)
-        return out
 
-    # -- measurement --------------------------------------------------------------------------------------------
-    KERNELS = {"ffn_gate_up": 0, "ffn_down": 1, "qkv_rope": 2, "attn_out": 3, "lm_head": 4, "attention": 5}
+class PlannedModel(CausalModel):
+    """A model whose config.json lists its layers (nfai_model_load_dir): dtype "bf16" serves it in bfloat16 with float32
+    where the design asks for it, "f32" runs everything in true 32-bit."""
 
-    def profile_kernel(self, which: str, iters: int) -> Tuple[float, int]:
-        ms = C.c_float()
-        nbytes = C.c_uint64()
-        check(self._lib.nfai_profile_kernel(self.handle, self.KERNELS[which], iters, C.byref(ms), C.byref(nbytes)),
-              self.ctx.handle)
-        return ms.value, nbytes.value
+    def __init__(self, ctx: CudaContext, path: str, context_size: int = 1024, dtype: str = "bf16"):
+        self.ctx = ctx
+        self._lib = _lib.load()
+        with open(os.path.join(path, "config.json")) as fh:
+            self.config = json.load(fh)
+        h = C.c_void_p()
+        check(self._lib.nfai_model_load_dir(ctx.handle, path.encode(), int(context_size), _dtype_code(dtype), C.byref(h)),
+              ctx.handle)
+        self._adopt(h, os.path.basename(os.path.normpath(path)))
 
-    def tune(self, which: str, mode: int, rows_per_warp: int, depth: int, ctas_per_sm: int):
-        check(self._lib.nfai_model_tune(self.handle, self.KERNELS[which], mode, rows_per_warp, depth, ctas_per_sm),
-              self.ctx.handle)
-
-    def set_prefetch(self, lookahead_bytes: int, extra_bytes: int = 0, mode: int = 1):
-        check(self._lib.nfai_model_set_prefetch(self.handle, int(lookahead_bytes), int(extra_bytes), mode),
-              self.ctx.handle)
-
-    def step_launches(self) -> int:
-        n = C.c_int()
-        check(self._lib.nfai_step_launches(self.handle, C.byref(n)), self.ctx.handle)
-        return n.value
-
-    def Dispose(self):
-        if getattr(self, "handle", None):
-            self._lib.nfai_model_destroy(self.handle)
-            self.handle = None
-
-    def __del__(self):
+    @classmethod
+    def from_tensors(cls, ctx: CudaContext, config: Dict[str, object], tensors: Iterable[Tuple[str, np.ndarray, int]],
+                     context_size: int = 1024, dtype: str = "bf16") -> "PlannedModel":
+        """From tensors in memory: (name, array, element code); a bfloat16 array holds its bits as uint16."""
+        self = cls.__new__(cls)
+        self.ctx = ctx
+        self._lib = _lib.load()
+        self.config = config
+        text = json.dumps(config).encode()
+        h = C.c_void_p()
+        check(self._lib.nfai_model_create_from_config(ctx.handle, text, len(text), int(context_size), _dtype_code(dtype),
+                                                      C.byref(h)), ctx.handle)
+        self.handle = h
         try:
-            self.Dispose()
+            for name, a, code in tensors:
+                a = np.ascontiguousarray(a)
+                ne = (C.c_uint64 * a.ndim)(*reversed(a.shape))
+                check(self._lib.nfai_model_tensor_begin(h, name.encode(), code, ne, a.ndim), ctx.handle)
+                check(self._lib.nfai_model_tensor_chunk(h, a.ctypes.data_as(C.c_void_p), a.nbytes), ctx.handle)
+                check(self._lib.nfai_model_tensor_end(h), ctx.handle)
+            check(self._lib.nfai_model_finalize(h), ctx.handle)
         except Exception:
-            pass
+            self.Dispose()
+            raise
+        self._adopt(h, str(config["architecture"]))
+        return self
+
+    def _adopt(self, handle, name: str):
+        self.handle = handle
+        self.hp = HParams()
+        check(self._lib.nfai_model_get_hparams(handle, C.byref(self.hp)), self.ctx.handle)
+        self.V, self.H, self.L = self.hp.V, self.hp.H, self.hp.L
+        self.weight_dtype = self.kv_dtype = _dtype_name(self.hp.weight_dtype)
+        self.ModelName = name
+
+    KERNELS = {"ffn_gate_up": 0, "ffn_down": 1, "latent_in": 2, "latent_out": 3, "lm_head": 4, "latent_attention": 5,
+               "ssm_in": 6, "ssm_step": 7, "ssm_out": 8}
+
+    def read_latent(self, layer: int, pos: int) -> Tuple[np.ndarray, np.ndarray]:
+        """Cached latent and rotated key part of one position of a latent attention layer."""
+        m = self.config["layers"][layer]["mixer"]
+        c, kr = np.empty(m["kv_rank"], np.float32), np.empty(m["rot_dim"], np.float32)
+        check(self._lib.nfai_read_kv(self.handle, layer, pos, self._fp(c), self._fp(kr)), self.ctx.handle)
+        return c, kr
+
+
+def config_tensors(config: Dict[str, object]) -> Dict[str, Tuple[int, ...]]:
+    """Names and shapes (outermost first) of the tensors a layer-plan configuration needs; raises for a configuration the
+    library does not accept. Needs no device."""
+    lib = _lib.load()
+    text = json.dumps(config).encode()
+    n = C.c_size_t()
+    check(lib.nfai_config_probe(text, len(text), None, None, 0, C.byref(n), None, 0))
+    buf = C.create_string_buffer(n.value + 1)
+    check(lib.nfai_config_probe(text, len(text), None, buf, n.value + 1, None, None, 0))
+    out = {}
+    for line in buf.value.decode().splitlines():
+        name, *dims = line.split()
+        out[name] = tuple(int(d) for d in dims)
+    return out
 
 
 class KvSnapshot:
     """Handle of nfai_kv_snapshot_*: belongs to one model, close() it before the model."""
 
-    def __init__(self, model: "LlamaModel", handle):
+    def __init__(self, model: "CausalModel", handle):
         self.model, self.handle = model, handle
 
     @property
     def position(self) -> int:
         return int(self.model._lib.nfai_kv_snapshot_position(self.handle))
 
-    def restore(self, model: Optional["LlamaModel"] = None):
+    def restore(self, model: Optional["CausalModel"] = None):
         m = model or self.model
         check(m._lib.nfai_kv_snapshot_restore(m.handle, self.handle), m.ctx.handle)
 

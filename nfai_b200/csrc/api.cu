@@ -13,43 +13,15 @@
 #include <string>
 #include <vector>
 
-#include "../../include/nfai_cuda.h"
-#include "kernels.h"
-#include "gemm_tc.h"
-#include "tp.h"
+#include "model.h"
 
 using namespace nfai;
 
 namespace {
-
 thread_local std::string g_err;  // failures of calls that have no context
-
-constexpr size_t kStageBytes = 16u << 20;
-constexpr int kStageSlots = 2;
-
-size_t align_up(size_t v, size_t a) { return (v + a - 1) / a * a; }
-size_t dtype_size(int dt) { return dt == NFAI_F16 ? 2 : 4; }
-
 }  // namespace
 
-struct nfai_ctx {
-  int device = 0;
-  int rank = 0, world = 1;
-  cudaStream_t stream = nullptr;
-  cudaEvent_t ev0 = nullptr, ev1 = nullptr;
-  void* stage[kStageSlots] = {nullptr, nullptr};  // pinned, device-visible
-  cudaEvent_t stage_ev[kStageSlots] = {nullptr, nullptr};
-  int stage_next = 0;
-  uint32_t* pin_small = nullptr;  // pinned scratch for tokens / state read-back (256 bytes)
-  uint32_t* dev_err = nullptr;    // device word for error bits of kernels that run outside a model step
-  TpComm* tp = nullptr;
-  bool pdl = true;
-  bool use_graph = true;
-  unsigned long long wait_ns = 1000000000ull;  // budget of every bounded device-side wait on peers (NFAI_WAIT_NS)
-  std::string err;
-};
-
-namespace {
+namespace nfai {
 
 int fail(nfai_ctx* c, int code, const char* fmt, ...) {
   char buf[512];
@@ -62,103 +34,12 @@ int fail(nfai_ctx* c, int code, const char* fmt, ...) {
   return code;
 }
 
-#define CU(c, call)                                                                                    \
-  do {                                                                                                 \
-    cudaError_t e__ = (call);                                                                          \
-    if (e__ != cudaSuccess)                                                                            \
-      return fail((c), e__ == cudaErrorMemoryAllocation ? NFAI_ERR_OOM : NFAI_ERR_CUDA, "%s: %s (%s:%d)", #call, \
-                  cudaGetErrorString(e__), __FILE__, __LINE__);                                        \
-  } while (0)
+int env_int(const char* name, int dflt) {
+  const char* v = getenv(name);
+  return v && *v ? atoi(v) : dflt;
+}
 
-struct Matrix {
-  void* ptr = nullptr;
-  uint64_t rows = 0, cols = 0;  // local (this rank's) shape
-  size_t bytes = 0;
-};
-
-struct Gain {
-  float* ptr = nullptr;
-  bool done = false;
-};
-
-struct LayerW {
-  Matrix qkv, o, gateup, down;
-  Gain attn_norm, ffn_norm;
-  bool got_q = false, got_k = false, got_v = false, got_o = false, got_gate = false, got_up = false, got_down = false;
-};
-
-// Where the tensor being uploaded goes.
-struct UploadTarget {
-  bool active = false;
-  bool skip = false;  // accepted and ignored (output.weight on a tied model)
-  std::string name;
-  int src_dtype = 0, dst_dtype = 0;
-  uint64_t K = 0, N = 0;  // source shape: N rows of K
-  uint64_t received = 0;  // source elements so far
-  IngestParams ip;
-  bool* done_flag = nullptr;
-};
-
-}  // namespace
-
-struct nfai_model {
-  nfai_ctx* ctx = nullptr;
-  nfai_hparams hp{};
-  // local (per-rank) geometry
-  uint32_t qHl = 0, kvHl = 0, qDimL = 0, kvDimL = 0, Fl = 0, Vl = 0, v_lo = 0;
-  bool finalized = false;
-  char* warena = nullptr;
-  size_t warena_bytes = 0;
-  Matrix embd, head;
-  bool got_embd = false, got_head = false;
-  Gain out_norm;
-  std::vector<LayerW> layers;
-  UploadTarget up;
-  // run-time buffers (one allocation)
-  char* rarena = nullptr;
-  void* kc = nullptr;
-  void* vc = nullptr;  // [L][ctx][kvDimL]
-  float2* rope_cs = nullptr;
-  float* xbuf = nullptr;  // [(2L+1)][H]: x_in(0), then per layer (after attention, after FFN)
-  float* q = nullptr;
-  float* attn_out = nullptr;
-  float* hbuf = nullptr;
-  float* logits = nullptr;
-  float* part_val = nullptr;
-  uint32_t* part_idx = nullptr;
-  uint32_t nparts = 0, nparts_alloc = 0;
-  float* attn_part = nullptr;
-  uint32_t* tickets = nullptr;
-  uint32_t S_max = 1;
-  uint32_t attn_heads = 4;  // query heads per attention CTA in the decode step
-  std::vector<AttnTileMaps> attn_maps;  // per layer, when the decode step uses the tile-staged attention kernel
-  bool attn_mma = false;                // long float16 caches: the tensor-core attention kernel (default over the tile-staged one)
-  StepState* state = nullptr;
-  uint32_t* history = nullptr;
-  uint32_t* prompt = nullptr;
-  float* pin_logits = nullptr;  // pinned V floats
-  float* tp_buf = nullptr;      // [H] partial sums exchanged between ranks
-  void* sample_scratch = nullptr;  // per-slice sums and candidates of the on-device sampler
-  cudaGraphExec_t g_full = nullptr, g_nohead = nullptr;
-  int launches_full = 0;
-  uint32_t pos = 0;  // host mirror of state->pos
-  GemvTune tune_qkv, tune_o, tune_gateup, tune_down, tune_head;
-  // batched prompt path (float16 weights, one GPU): chunk workspace
-  bool prefill_gemm = false;
-  uint32_t pf_chunk = 0;
-  float* pfX0 = nullptr;      // [chunk][H] residual stream
-  float* pfX1 = nullptr;      // [chunk][H]
-  __half* pfA = nullptr;      // [chunk][max(H, qDim)] normalised activations
-  float* pfQ = nullptr;       // [chunk][qDim] rotated queries
-  __half* pfAO = nullptr;     // [chunk][qDim] attention output
-  __half* pfH = nullptr;      // [chunk][F] SiLU(gate)*up
-  float* pfPart = nullptr;    // split-K partial tiles of the prompt GEMMs
-  size_t pfPartFloats = 0;
-  uint32_t* pfTok = nullptr;  // [chunk]
-  // L2 look-ahead: how far beyond the weights a kernel consumes the step's weight sequence is requested
-  uint64_t pf_look = 0, pf_extra = 0;
-  int pf_mode = 1;
-};
+}  // namespace nfai
 
 namespace {
 
@@ -167,17 +48,14 @@ float* x_mid(nfai_model* m, uint32_t layer) { return m->xbuf + (size_t)(2 * laye
 
 size_t kv_layer_elems(const nfai_model* m) { return (size_t)m->hp.ctx * m->kvDimL; }
 
-int env_int(const char* name, int dflt) {
-  const char* v = getenv(name);
-  return v && *v ? atoi(v) : dflt;
-}
-
 bool ring_wanted(uint32_t positions) {
   const int v = env_int("NFAI_ATTN_RING", -1);
   return v < 0 ? positions > 4096 : v != 0;
 }
 
-void read_tune(const char* name, GemvTune& t, int r_default, int u_default) {
+}  // namespace
+
+void nfai::read_tune(const char* name, GemvTune& t, int r_default, int u_default) {
   t.rows_per_warp = r_default;
   t.unroll = u_default;
   std::string key = std::string("NFAI_TUNE_") + name;
@@ -196,6 +74,8 @@ void read_tune(const char* name, GemvTune& t, int r_default, int u_default) {
     }
   }
 }
+
+namespace {
 
 // ---- the decode step as a sequence of launches (captured into a graph or run eagerly) -------------------------
 GemvParams qkv_params(nfai_model* m, uint32_t l) {
@@ -362,6 +242,7 @@ PrefetchPlanner make_planner(nfai_model* m, bool with_head) {
 }
 
 cudaError_t record_step(nfai_model* m, bool with_head, bool from_prompt, int* launches) {
+  if (m->plan) return plan_record_step(m, with_head, from_prompt, launches);
   nfai_ctx* c = m->ctx;
   const nfai_hparams& hp = m->hp;
   cudaStream_t s = c->stream;
@@ -428,7 +309,7 @@ cudaError_t record_step(nfai_model* m, bool with_head, bool from_prompt, int* la
     GemvParams gg = gateup_params(m, l);
     gg.pf = pp.next(end_of(LW.gateup), true);
     pull_into(gg, 2 * l, x_in(m, l), x_mid(m, l));
-    STEP(launch_gemv(s, wdt, kvdt, EPI_SILU_MUL, gg, m->tune_gateup, pdl_x));
+    STEP(launch_gemv(s, wdt, kvdt, EPI_GATED, gg, m->tune_gateup, pdl_x));
     GemvParams gd = down_params(m, l);
     gd.pf = pp.next(pp.off(LW.ffn_norm.ptr) + (uint64_t)hp.H * 4, true);
     push_from(gd, 2 * l + 1);
@@ -498,7 +379,9 @@ int run_step(nfai_model* m, bool with_head, bool from_prompt) {
   return NFAI_OK;
 }
 
-int check_state(nfai_model* m, StepState* host_copy) {
+}  // namespace
+
+int nfai::check_state(nfai_model* m, StepState* host_copy) {
   nfai_ctx* c = m->ctx;
   CU(c, cudaMemcpyAsync(c->pin_small, m->state, sizeof(StepState), cudaMemcpyDeviceToHost, c->stream));
   CU(c, cudaStreamSynchronize(c->stream));
@@ -515,13 +398,70 @@ int check_state(nfai_model* m, StepState* host_copy) {
   return NFAI_OK;
 }
 
-int set_state_word(nfai_model* m, size_t offset, uint32_t value, int slot) {
+int nfai::set_state_word(nfai_model* m, size_t offset, uint32_t value, int slot) {
   nfai_ctx* c = m->ctx;
   // the copy reads the pinned word when it executes: every copy that may still be pending has its own slot
   c->pin_small[32 + slot] = value;
   CU(c, cudaMemcpyAsync((char*)m->state + offset, &c->pin_small[32 + slot], 4, cudaMemcpyHostToDevice, c->stream));
   return NFAI_OK;
 }
+
+// Both decode graphs (with and without LM head), replacing what the model had; on failure the old ones stay.
+int nfai::capture_graphs(nfai_model* m) {
+  nfai_ctx* c = m->ctx;
+  if (!c->use_graph) {
+    m->launches_full = m->plan ? plan_step_launches(m) : 3 + 5 * (int)m->hp.L;
+    return NFAI_OK;
+  }
+  cudaGraphExec_t gf = nullptr, gn = nullptr;
+  int launches = 0;
+  int rc = capture(m, true, false, &gf, &launches);
+  if (rc == NFAI_OK) rc = capture(m, false, true, &gn, nullptr);
+  if (rc != NFAI_OK) {
+    if (gf) cudaGraphExecDestroy(gf);
+    return rc;
+  }
+  if (m->g_full) cudaGraphExecDestroy(m->g_full);
+  if (m->g_nohead) cudaGraphExecDestroy(m->g_nohead);
+  m->g_full = gf;
+  m->g_nohead = gn;
+  m->launches_full = launches;
+  return NFAI_OK;
+}
+
+CommonOffsets nfai::place_common(nfai_model* m, Arena& a) {
+  CommonOffsets o;
+  // arg-max partials: room for every launch shape nfai_model_tune may select later (up to 16 CTAs per SM)
+  m->nparts_alloc = sm_count() * 16;
+  o.logits = a.take((size_t)m->Vl * 4);
+  o.part_val = a.take((size_t)m->nparts_alloc * 4);
+  o.part_idx = a.take((size_t)m->nparts_alloc * 4);
+  o.state = a.take(sizeof(StepState));
+  o.history = a.take((size_t)m->hp.ctx * 4);
+  o.prompt = a.take((size_t)m->hp.ctx * 4);
+  o.sample = a.take(sample_scratch_bytes(m->Vl, nullptr));
+  return o;
+}
+
+void nfai::bind_common(nfai_model* m, const CommonOffsets& o) {
+  m->logits = (float*)(m->rarena + o.logits);
+  m->part_val = (float*)(m->rarena + o.part_val);
+  m->part_idx = (uint32_t*)(m->rarena + o.part_idx);
+  m->state = (StepState*)(m->rarena + o.state);
+  m->history = (uint32_t*)(m->rarena + o.history);
+  m->prompt = (uint32_t*)(m->rarena + o.prompt);
+  m->sample_scratch = m->rarena + o.sample;
+}
+
+int nfai::ready(nfai_model* m) {
+  if (!m) return fail(nullptr, NFAI_ERR_ARG, "model is null");
+  if (!m->finalized) return fail(m->ctx, NFAI_ERR_STATE, "model is not finalized");
+  cudaError_t e = cudaSetDevice(m->ctx->device);
+  if (e != cudaSuccess) return fail(m->ctx, NFAI_ERR_CUDA, "cudaSetDevice: %s", cudaGetErrorString(e));
+  return NFAI_OK;
+}
+
+namespace {
 
 // ---- tensor name -> destination -----------------------------------------------------------------------------
 int resolve_target(nfai_model* m, const char* name, int src_dtype, const uint64_t* shape, int ndim, UploadTarget* t) {
@@ -832,10 +772,12 @@ int nfai_model_tensor_begin(nfai_model* m, const char* name, int src_dtype, cons
   if (m->finalized) return fail(c, NFAI_ERR_STATE, "model already finalized");
   if (m->up.active) return fail(c, NFAI_ERR_STATE, "tensor %s is still open", m->up.name.c_str());
   if (!name || !shape || ndim < 1 || ndim > 2) return fail(c, NFAI_ERR_ARG, "bad tensor description");
-  if (src_dtype != NFAI_F32 && src_dtype != NFAI_F16) return fail(c, NFAI_ERR_ARG, "source dtype must be NFAI_F32 or NFAI_F16");
+  if (src_dtype != NFAI_F32 && src_dtype != NFAI_F16 && src_dtype != NFAI_BF16)
+    return fail(c, NFAI_ERR_ARG, "source dtype must be NFAI_F32, NFAI_F16 or NFAI_BF16");
   UploadTarget t;
-  int rc = resolve_target(m, name, src_dtype, shape, ndim, &t);
+  int rc = m->plan ? plan_resolve(m, name, shape, ndim, &t) : resolve_target(m, name, src_dtype, shape, ndim, &t);
   if (rc) return rc;
+  t.src_dtype = src_dtype;
   t.active = true;
   m->up = t;
   return NFAI_OK;
@@ -893,6 +835,7 @@ int nfai_model_finalize(nfai_model* m) {
   nfai_ctx* c = m->ctx;
   if (m->finalized) return fail(c, NFAI_ERR_STATE, "model already finalized");
   if (m->up.active) return fail(c, NFAI_ERR_STATE, "tensor %s is still open", m->up.name.c_str());
+  if (m->plan) return plan_finalize(m);
   const nfai_hparams& hp = m->hp;
   if (!m->got_embd || !m->out_norm.done || (!hp.tied && !m->got_head)) return fail(c, NFAI_ERR_STATE, "missing token_embd / output_norm / output tensors");
   for (uint32_t l = 0; l < hp.L; ++l) {
@@ -911,8 +854,8 @@ int nfai_model_finalize(nfai_model* m) {
   if (m->attn_heads != 1 && m->attn_heads != 2 && m->attn_heads != 4) m->attn_heads = kAttnHeadsPerCta;
   m->S_max = attn_splits(m->qHl, m->kvHl, hp.ctx, m->attn_heads, kAttnMinChunk);
   const size_t kvs = dtype_size(hp.kv_dtype);
-  size_t off = 0;
-  auto take = [&](size_t bytes) { size_t o = off; off = align_up(off + bytes, 256); return o; };
+  Arena arena;
+  auto take = [&](size_t bytes) { return arena.take(bytes); };
   const size_t o_kc = take((size_t)hp.L * kv_layer_elems(m) * kvs);
   const size_t o_vc = take((size_t)hp.L * kv_layer_elems(m) * kvs);
   const size_t o_rope = take((size_t)hp.ctx * (hp.ropeDim / 2) * sizeof(float2) + 16);
@@ -920,18 +863,10 @@ int nfai_model_finalize(nfai_model* m) {
   const size_t o_q = take((size_t)m->qDimL * 4);
   const size_t o_ao = take((size_t)m->qDimL * 4);
   const size_t o_h = take((size_t)m->Fl * 4);
-  const size_t o_lg = take((size_t)m->Vl * 4);
-  // room for every launch shape nfai_model_tune may select later (up to 16 CTAs per SM)
-  const size_t npart_alloc = (size_t)sm_count() * 16;
-  m->nparts_alloc = (uint32_t)npart_alloc;
-  const size_t o_pv = take(npart_alloc * 4);
-  const size_t o_pi = take(npart_alloc * 4);
+  const CommonOffsets common = place_common(m, arena);
   const uint32_t S_alloc = m->S_max;
   const size_t o_ap = take(attn_part_floats(m->qHl, hp.d, S_alloc) * 4);
   const size_t o_tk = take((size_t)m->qHl * 4);  // one ticket per (kv head, head group); at most one per query head
-  const size_t o_st = take(sizeof(StepState));
-  const size_t o_hi = take((size_t)hp.ctx * 4);
-  const size_t o_pr = take((size_t)hp.ctx * 4);
   const size_t o_tp = take((size_t)hp.H * 4);
   // batched prompt workspace
   const bool want_pf = hp.weight_dtype == NFAI_F16 && env_int("NFAI_PREFILL_GEMM", 1) != 0 &&
@@ -952,7 +887,7 @@ int nfai_model_finalize(nfai_model* m) {
   // split-K happens only below 120 output tiles of 128 x 128, with at most one CTA per SM: that many tiles of partials bound it
   const size_t pf_part_floats = want_pf && env_int("NFAI_GEMM_SPLIT", 1) ? (size_t)sm_count() * 128 * 128 * 2 : 0;
   const size_t o_pp = take(pf_part_floats * 4);
-  const size_t o_ss = take(sample_scratch_bytes(m->Vl, nullptr));
+  const size_t off = arena.off;
   cudaError_t e = cudaMalloc((void**)&m->rarena, off);
   if (e != cudaSuccess) return fail(c, NFAI_ERR_OOM, "cudaMalloc of %zu run-time bytes (KV cache etc.): %s", off, cudaGetErrorString(e));
   CU(c, cudaMemsetAsync(m->rarena, 0, off, c->stream));
@@ -971,19 +906,14 @@ int nfai_model_finalize(nfai_model* m) {
       }
     }
   }
+  bind_common(m, common);
   m->rope_cs = (float2*)(m->rarena + o_rope);
   m->xbuf = (float*)(m->rarena + o_x);
   m->q = (float*)(m->rarena + o_q);
   m->attn_out = (float*)(m->rarena + o_ao);
   m->hbuf = (float*)(m->rarena + o_h);
-  m->logits = (float*)(m->rarena + o_lg);
-  m->part_val = (float*)(m->rarena + o_pv);
-  m->part_idx = (uint32_t*)(m->rarena + o_pi);
   m->attn_part = (float*)(m->rarena + o_ap);
   m->tickets = (uint32_t*)(m->rarena + o_tk);
-  m->state = (StepState*)(m->rarena + o_st);
-  m->history = (uint32_t*)(m->rarena + o_hi);
-  m->prompt = (uint32_t*)(m->rarena + o_pr);
   m->tp_buf = (float*)(m->rarena + o_tp);
   m->prefill_gemm = want_pf && pfc > 0;
   m->pf_chunk = pfc;
@@ -996,7 +926,6 @@ int nfai_model_finalize(nfai_model* m) {
   m->pfTok = (uint32_t*)(m->rarena + o_pt);
   m->pfPart = pf_part_floats ? (float*)(m->rarena + o_pp) : nullptr;
   m->pfPartFloats = pf_part_floats;
-  m->sample_scratch = m->rarena + o_ss;
   // RoPE table on the host, float32, as the reference builds its frequency table
   // (NFAI.Vulkan.Shaders/TransformerBlock.cs:33-38) and its shader forms theta = f[m] * float(pos)
   // (NFAI.Vulkan.Shaders/RoPEShader.cs:252-254); cos/sin from the host libm.
@@ -1014,14 +943,8 @@ int nfai_model_finalize(nfai_model* m) {
   }
   CU(c, cudaHostAlloc((void**)&m->pin_logits, (size_t)hp.V * 4, cudaHostAllocDefault));
   CU(c, cudaStreamSynchronize(c->stream));
-  if (c->use_graph) {
-    int rc = capture(m, true, false, &m->g_full, &m->launches_full);
-    if (rc) return rc;
-    rc = capture(m, false, true, &m->g_nohead, nullptr);
-    if (rc) return rc;
-  } else {
-    m->launches_full = 3 + 5 * (int)hp.L;
-  }
+  int rc = capture_graphs(m);
+  if (rc) return rc;
   m->pos = 0;
   m->finalized = true;
   return NFAI_OK;
@@ -1038,14 +961,6 @@ int nfai_model_destroy(nfai_model* m) {
   if (m->rarena) cudaFree(m->rarena);
   if (m->warena) cudaFree(m->warena);
   delete m;
-  return NFAI_OK;
-}
-
-static int ready(nfai_model* m) {
-  if (!m) return fail(nullptr, NFAI_ERR_ARG, "model is null");
-  if (!m->finalized) return fail(m->ctx, NFAI_ERR_STATE, "model is not finalized");
-  cudaError_t e = cudaSetDevice(m->ctx->device);
-  if (e != cudaSuccess) return fail(m->ctx, NFAI_ERR_CUDA, "cudaSetDevice: %s", cudaGetErrorString(e));
   return NFAI_OK;
 }
 
@@ -1125,7 +1040,7 @@ static int prefill_batched(nfai_model* m, const uint32_t* tokens, int n) {
       if (tp_on) CU(c, tp_allreduce(c->tp, s, m->pfX1, (size_t)T * hp.H));
       CU(c, launch_rmsnorm_to_half(s, m->pfX1, L.ffn_norm.ptr, hp.eps, T, hp.H, m->pfA, tp_on));
       GemmEpilogue eg;
-      eg.kind = GEMM_EPI_SILU_MUL; eg.out_f16 = m->pfH;
+      eg.kind = GEMM_EPI_GATED; eg.out_act = m->pfH;
       eg.scratch = m->pfPart; eg.scratch_floats = m->pfPartFloats;
       CU(c, launch_gemm_tc(s, m->pfA, (const __half*)L.gateup.ptr, T, 2 * m->Fl, hp.H, eg, err));
       GemmEpilogue ed;
@@ -1172,6 +1087,9 @@ static int prefill_batched(nfai_model* m, const uint32_t* tokens, int n) {
   return NFAI_OK;
 }
 
+// Fewer tokens than this go through the decode step one by one.
+static constexpr int kMinBatch = 8;
+
 int nfai_prefill(nfai_model* m, const uint32_t* tokens, int n, float* logits_last, uint32_t* argmax_last) {
   int rc = ready(m);
   if (rc) return rc;
@@ -1181,8 +1099,8 @@ int nfai_prefill(nfai_model* m, const uint32_t* tokens, int n, float* logits_las
     return fail(c, NFAI_ERR_CONTEXT_FULL, "prompt of %d tokens at position %u exceeds the KV-cache capacity %u", n, m->pos, m->hp.ctx);
   for (int i = 0; i < n; ++i)
     if (tokens[i] >= m->hp.V) return fail(c, NFAI_ERR_ARG, "token id %u out of range (V = %u)", tokens[i], m->hp.V);
-  if (m->prefill_gemm && n >= 8) {
-    if ((rc = prefill_batched(m, tokens, n))) return rc;
+  if (m->plan ? plan_batched(m) && n >= kMinBatch : m->prefill_gemm && n >= kMinBatch) {
+    if ((rc = m->plan ? plan_prefill(m, tokens, n, nullptr, 0, nullptr) : prefill_batched(m, tokens, n))) return rc;
     m->pos += (uint32_t)n;
     return fetch_outputs(m, logits_last, argmax_last);
   }
@@ -1196,6 +1114,33 @@ int nfai_prefill(nfai_model* m, const uint32_t* tokens, int n, float* logits_las
   if ((rc = run_step(m, true, false))) return rc;
   m->pos += (uint32_t)n;
   return fetch_outputs(m, logits_last, argmax_last);
+}
+
+int nfai_forward(nfai_model* m, const uint32_t* tokens, int n, const uint32_t* want, int n_want, float* logits) {
+  int rc = ready(m);
+  if (rc) return rc;
+  nfai_ctx* c = m->ctx;
+  if (!tokens || n <= 0) return fail(c, NFAI_ERR_ARG, "no tokens");
+  if (n_want < 0 || (n_want && (!want || !logits))) return fail(c, NFAI_ERR_ARG, "wanted places without a list or an output");
+  for (int i = 0; i < n_want; ++i)
+    if (want[i] >= (uint32_t)n || (i && want[i] <= want[i - 1])) return fail(c, NFAI_ERR_ARG, "wanted places must be ascending and below n");
+  if (m->plan && plan_batched(m) && n >= kMinBatch && n_want > 0 && !(n_want == 1 && want[0] == (uint32_t)n - 1)) {
+    if ((uint64_t)m->pos + (uint64_t)n > m->hp.ctx)
+      return fail(c, NFAI_ERR_CONTEXT_FULL, "%d tokens at position %u exceed the KV-cache capacity %u", n, m->pos, m->hp.ctx);
+    for (int i = 0; i < n; ++i)
+      if (tokens[i] >= m->hp.V) return fail(c, NFAI_ERR_ARG, "token id %u out of range (V = %u)", tokens[i], m->hp.V);
+    if ((rc = plan_prefill(m, tokens, n, want, n_want, logits))) return rc;
+    m->pos += (uint32_t)n;
+    return fetch_outputs(m, nullptr, nullptr);
+  }
+  // a portion ends behind every wanted place: its last logits are the ones asked for
+  int done = 0;
+  for (int i = 0; i < n_want; ++i) {
+    const int end = (int)want[i] + 1;
+    if ((rc = nfai_prefill(m, tokens + done, end - done, logits + (size_t)i * m->hp.V, nullptr))) return rc;
+    done = end;
+  }
+  return done < n ? nfai_prefill(m, tokens + done, n - done, nullptr, nullptr) : NFAI_OK;
 }
 
 int nfai_decode_greedy(nfai_model* m, uint32_t first_token, int n_steps, uint32_t* out_tokens, float* elapsed_ms) {
@@ -1289,6 +1234,9 @@ int nfai_set_position(nfai_model* m, uint32_t pos) {
   int rc = ready(m);
   if (rc) return rc;
   if (pos > m->hp.ctx) return fail(m->ctx, NFAI_ERR_ARG, "position beyond the KV-cache capacity");
+  // recurrent states cannot be rewound: only the start (states begin at zero there) and the current position
+  if (m->plan && pos != 0 && pos != m->pos)
+    return fail(m->ctx, NFAI_ERR_STATE, "a model with recurrent layers can only return to position 0; use a snapshot");
   if ((rc = set_state_word(m, offsetof(StepState, pos), pos, 3))) return rc;
   CU(m->ctx, cudaStreamSynchronize(m->ctx->stream));
   m->pos = pos;
@@ -1306,7 +1254,8 @@ struct nfai_kv_snapshot {
   int device = 0;
   uint32_t pos = 0, cur_token = 0, last_argmax = 0;
   char* dev = nullptr;
-  size_t row_bytes = 0;  // bytes of K (or V) of one layer: pos * kvDim * element size
+  size_t row_bytes = 0;    // bytes of K (or V) of one layer: pos * kvDim * element size
+  size_t state_bytes = 0;  // everything in front of the logits
 };
 
 extern "C" {
@@ -1326,13 +1275,15 @@ int nfai_kv_snapshot_create(nfai_model* m, nfai_kv_snapshot** out) {
   s->pos = m->pos;
   s->cur_token = st.cur_token;
   s->last_argmax = st.last_argmax;
-  s->row_bytes = (size_t)m->pos * m->kvDimL * kvs;
-  const size_t total = 2 * (size_t)hp.L * s->row_bytes + (size_t)m->Vl * 4;
+  s->row_bytes = m->plan ? 0 : (size_t)m->pos * m->kvDimL * kvs;
+  s->state_bytes = m->plan ? plan_snapshot_bytes(m, m->pos) : 2 * (size_t)hp.L * s->row_bytes;
+  const size_t total = s->state_bytes + (size_t)m->Vl * 4;
   cudaError_t e = cudaMalloc((void**)&s->dev, total);
   if (e != cudaSuccess) {
     delete s;
     return fail(c, NFAI_ERR_OOM, "cudaMalloc of %zu snapshot bytes: %s", total, cudaGetErrorString(e));
   }
+  if (m->plan) e = plan_snapshot_copy(m, m->pos, s->dev, true);
   for (uint32_t l = 0; l < hp.L && e == cudaSuccess; ++l) {
     const size_t lo = (size_t)l * kv_layer_elems(m) * kvs;
     if (s->row_bytes) {
@@ -1342,7 +1293,7 @@ int nfai_kv_snapshot_create(nfai_model* m, nfai_kv_snapshot** out) {
     }
   }
   if (e == cudaSuccess)
-    e = cudaMemcpyAsync(s->dev + 2 * (size_t)hp.L * s->row_bytes, m->logits, (size_t)m->Vl * 4, cudaMemcpyDeviceToDevice, c->stream);
+    e = cudaMemcpyAsync(s->dev + s->state_bytes, m->logits, (size_t)m->Vl * 4, cudaMemcpyDeviceToDevice, c->stream);
   if (e == cudaSuccess) e = cudaStreamSynchronize(c->stream);
   if (e != cudaSuccess) {
     cudaFree(s->dev);
@@ -1361,6 +1312,7 @@ int nfai_kv_snapshot_restore(nfai_model* m, const nfai_kv_snapshot* s) {
   const nfai_hparams& hp = m->hp;
   const size_t kvs = dtype_size(hp.kv_dtype);
   CU(c, cudaSetDevice(c->device));
+  if (m->plan) CU(c, plan_snapshot_copy(m, s->pos, s->dev, false));
   for (uint32_t l = 0; l < hp.L; ++l) {
     const size_t lo = (size_t)l * kv_layer_elems(m) * kvs;
     if (s->row_bytes) {
@@ -1368,7 +1320,7 @@ int nfai_kv_snapshot_restore(nfai_model* m, const nfai_kv_snapshot* s) {
       CU(c, cudaMemcpyAsync((char*)m->vc + lo, s->dev + (2 * (size_t)l + 1) * s->row_bytes, s->row_bytes, cudaMemcpyDeviceToDevice, c->stream));
     }
   }
-  CU(c, cudaMemcpyAsync(m->logits, s->dev + 2 * (size_t)hp.L * s->row_bytes, (size_t)m->Vl * 4, cudaMemcpyDeviceToDevice, c->stream));
+  CU(c, cudaMemcpyAsync(m->logits, s->dev + s->state_bytes, (size_t)m->Vl * 4, cudaMemcpyDeviceToDevice, c->stream));
   if ((rc = set_state_word(m, offsetof(StepState, pos), s->pos, 3))) return rc;
   if ((rc = set_state_word(m, offsetof(StepState, cur_token), s->cur_token, 4))) return rc;
   if ((rc = set_state_word(m, offsetof(StepState, last_argmax), s->last_argmax, 5))) return rc;
@@ -1391,6 +1343,10 @@ static int kv_rw(nfai_model* m, uint32_t layer, uint32_t pos, float* k, float* v
   int rc = ready(m);
   if (rc) return rc;
   nfai_ctx* c = m->ctx;
+  if (m->plan) {
+    if (kin || vin) return fail(c, NFAI_ERR_STATE, "the caches of a layer-plan model cannot be overwritten");
+    return plan_read_kv(m, layer, pos, k, v);
+  }
   if (layer >= m->hp.L || pos >= m->hp.ctx) return fail(c, NFAI_ERR_ARG, "layer or position out of range");
   const size_t kvs = dtype_size(m->hp.kv_dtype);
   const size_t off = ((size_t)layer * kv_layer_elems(m) + (size_t)pos * m->kvDimL) * kvs;
@@ -1428,6 +1384,7 @@ int nfai_write_kv_range(nfai_model* m, uint32_t layer, uint32_t pos0, uint32_t n
   int rc = ready(m);
   if (rc) return rc;
   nfai_ctx* c = m->ctx;
+  if (m->plan) return fail(c, NFAI_ERR_STATE, "the caches of a layer-plan model cannot be overwritten");
   if (!k || !v || !n || layer >= m->hp.L || pos0 >= m->hp.ctx || n > m->hp.ctx - pos0)
     return fail(c, NFAI_ERR_ARG, "layer or position range out of bounds");
   const size_t kvs = dtype_size(m->hp.kv_dtype);
@@ -1453,6 +1410,7 @@ int nfai_read_hidden(nfai_model* m, uint32_t layer, float* out) {
   if (rc) return rc;
   nfai_ctx* c = m->ctx;
   if (layer >= m->hp.L || !out) return fail(c, NFAI_ERR_ARG, "layer out of range or null output");
+  if (m->plan) return plan_read_hidden(m, layer, out);
   CU(c, cudaStreamSynchronize(c->stream));
   CU(c, cudaMemcpy(out, x_in(m, layer + 1), (size_t)m->hp.H * 4, cudaMemcpyDeviceToHost));
   return NFAI_OK;
@@ -1490,7 +1448,7 @@ int nfai_model_tune(nfai_model* m, int which, int mode, int rows_per_warp, int d
   CU(c, cudaSetDevice(c->device));
   CU(c, cudaStreamSynchronize(c->stream));
   if (which == 4) {
-    GemvParams hp_ = head_params(m);
+    GemvParams hp_ = m->plan ? plan_head_params(m) : head_params(m);
     uint32_t np = gemv_grid(m->hp.weight_dtype, EPI_LOGITS, hp_, *t);
     if (np > m->nparts_alloc) {
       *t = old;
@@ -1498,49 +1456,23 @@ int nfai_model_tune(nfai_model* m, int which, int mode, int rows_per_warp, int d
     }
     m->nparts = np;
   }
-  if (c->use_graph) {
-    cudaGraphExec_t gf = nullptr, gn = nullptr;
-    int launches = 0;
-    int rc = capture(m, true, false, &gf, &launches);
-    if (rc == NFAI_OK) rc = capture(m, false, true, &gn, nullptr);
-    if (rc != NFAI_OK) {
-      if (gf) cudaGraphExecDestroy(gf);
-      *t = old;
-      return rc;
-    }
-    cudaGraphExecDestroy(m->g_full);
-    cudaGraphExecDestroy(m->g_nohead);
-    m->g_full = gf;
-    m->g_nohead = gn;
-    m->launches_full = launches;
-  }
-  return NFAI_OK;
+  int rc = capture_graphs(m);
+  if (rc != NFAI_OK) *t = old;
+  return rc;
 }
 
 int nfai_model_set_prefetch(nfai_model* m, uint64_t lookahead_bytes, uint64_t extra_bytes, int mode) {
   if (!m) return fail(nullptr, NFAI_ERR_ARG, "model is null");
   nfai_ctx* c = m->ctx;
   if (mode != 0 && mode != 1) return fail(c, NFAI_ERR_ARG, "mode must be 0 (per line) or 1 (bulk)");
+  if (m->plan) return fail(c, NFAI_ERR_STATE, "the L2 look-ahead is a feature of the Llama step");
   m->pf_look = lookahead_bytes;
   m->pf_extra = extra_bytes;
   m->pf_mode = mode;
   if (!m->finalized || !c->use_graph) return NFAI_OK;
   CU(c, cudaSetDevice(c->device));
   CU(c, cudaStreamSynchronize(c->stream));
-  cudaGraphExec_t gf = nullptr, gn = nullptr;
-  int launches = 0;
-  int rc = capture(m, true, false, &gf, &launches);
-  if (rc == NFAI_OK) rc = capture(m, false, true, &gn, nullptr);
-  if (rc != NFAI_OK) {
-    if (gf) cudaGraphExecDestroy(gf);
-    return rc;
-  }
-  cudaGraphExecDestroy(m->g_full);
-  cudaGraphExecDestroy(m->g_nohead);
-  m->g_full = gf;
-  m->g_nohead = gn;
-  m->launches_full = launches;
-  return NFAI_OK;
+  return capture_graphs(m);
 }
 
 int nfai_step_launches(const nfai_model* m, int* out) {
@@ -1554,21 +1486,28 @@ int nfai_profile_kernel(nfai_model* m, int which, int iters, float* avg_ms, uint
   if (rc) return rc;
   nfai_ctx* c = m->ctx;
   const nfai_hparams& hp = m->hp;
-  if (iters <= 0 || which < 0 || which > 5) return fail(c, NFAI_ERR_ARG, "bad kernel selector or iteration count");
+  if (iters <= 0 || which < 0 || which > (m->plan ? 8 : 5)) return fail(c, NFAI_ERR_ARG, "bad kernel selector or iteration count");
   if (which == 5 && m->pos == 0) return fail(c, NFAI_ERR_STATE, "attention profiling needs at least one cached position");
   const int wdt = hp.weight_dtype, kvdt = hp.kv_dtype;
   const size_t ws = dtype_size(wdt), kvs = dtype_size(kvdt);
   // the QKV kernel writes a cache row at state->pos: profile it one row below the current position
   uint32_t saved_pos = m->pos;
-  if (which == 2 && saved_pos >= hp.ctx) return fail(c, NFAI_ERR_CONTEXT_FULL, "QKV profiling needs one free cache row");
+  if ((which == 2 || m->plan) && saved_pos >= hp.ctx) return fail(c, NFAI_ERR_CONTEXT_FULL, "QKV profiling needs one free cache row");
   if (which == 5) {
     // attention reads positions 0..pos: make seq = pos (all of them written)
     if ((rc = set_state_word(m, offsetof(StepState, pos), saved_pos - 1, 3))) return rc;
   }
+  // launches of a state space step advance the state: keep it and put it back
+  struct Keep {
+    nfai_kv_snapshot* s = nullptr;
+    ~Keep() { nfai_kv_snapshot_destroy(s); }
+  } keep;
+  if (m->plan && (rc = nfai_kv_snapshot_create(m, &keep.s))) return rc;
   auto one = [&](int i) -> cudaError_t {
+    if (m->plan) return plan_profile_launch(m, which, i);
     uint32_t l = (uint32_t)i % hp.L;
     switch (which) {
-      case 0: return launch_gemv(c->stream, wdt, kvdt, EPI_SILU_MUL, gateup_params(m, l), m->tune_gateup, false);
+      case 0: return launch_gemv(c->stream, wdt, kvdt, EPI_GATED, gateup_params(m, l), m->tune_gateup, false);
       case 1: return launch_gemv(c->stream, wdt, kvdt, EPI_STORE, down_params(m, l), m->tune_down, false);
       case 2: return launch_gemv(c->stream, wdt, kvdt, EPI_QKV_ROPE, qkv_params(m, l), m->tune_qkv, false);
       case 3: return launch_gemv(c->stream, wdt, kvdt, EPI_STORE, o_params(m, l), m->tune_o, false);
@@ -1607,9 +1546,10 @@ int nfai_profile_kernel(nfai_model* m, int which, int iters, float* avg_ms, uint
   float ms = 0.f;
   CU(c, cudaEventElapsedTime(&ms, c->ev0, c->ev1));
   if (avg_ms) *avg_ms = ms / (float)iters;
+  if (keep.s && (rc = nfai_kv_snapshot_restore(m, keep.s))) return rc;
   if (bytes_per_launch) {
-    uint64_t b = 0;
-    switch (which) {
+    uint64_t b = m->plan ? plan_profile_bytes(m, which) : 0;
+    if (!m->plan) switch (which) {
       case 0: b = 2ull * m->Fl * hp.H * ws + (uint64_t)hp.H * 4; break;
       case 1: b = (uint64_t)hp.H * m->Fl * ws; break;
       case 2: b = (uint64_t)(m->qDimL + 2 * m->kvDimL) * hp.H * ws + (uint64_t)hp.H * 4 + 2ull * m->kvDimL * kvs; break;
@@ -1685,7 +1625,7 @@ int nfai_op_ffn_gate_up(nfai_ctx* c, const void* Wgu, int dtype, const float* x,
   p.W = Wgu; p.N = 2 * F; p.K = H; p.x = x; p.gain = gain; p.eps = eps; p.y = h_out;
   GemvTune t;
   read_tune("OP", t, 2, 4);
-  return op_end(c, launch_gemv(c->stream, dtype, NFAI_F32, EPI_SILU_MUL, p, t, false));
+  return op_end(c, launch_gemv(c->stream, dtype, NFAI_F32, EPI_GATED, p, t, false));
 }
 
 size_t nfai_op_attn_scratch_bytes(uint32_t qH, uint32_t kvH, uint32_t d, uint32_t max_seq) {

@@ -1,5 +1,6 @@
 // Shared device helpers for the sm_100a kernels of libnfai_cuda.
 #pragma once
+#include <cuda_bf16.h>
 #include <cuda_fp16.h>
 #include <cuda_runtime.h>
 #include <stdint.h>
@@ -105,6 +106,19 @@ struct WeightVec<__half> {
 };
 
 template <>
+struct WeightVec<__nv_bfloat16> {
+  static constexpr int kElems = 8;
+  __device__ __forceinline__ static void unpack(const uint4& v, float (&f)[8]) {
+    const uint32_t w[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {  // a bfloat16 is the upper half of a float32
+      f[2 * i] = __uint_as_float(w[i] << 16);
+      f[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
+    }
+  }
+};
+
+template <>
 struct WeightVec<float> {
   static constexpr int kElems = 4;
   __device__ __forceinline__ static void unpack(const uint4& v, float (&f)[4]) {
@@ -117,7 +131,17 @@ struct WeightVec<float> {
 
 __device__ __forceinline__ float to_float(float v) { return v; }
 __device__ __forceinline__ float to_float(__half v) { return __half2float(v); }
+__device__ __forceinline__ float to_float(__nv_bfloat16 v) { return __bfloat162float(v); }
 __device__ __forceinline__ void store_as(float* p, float v) { *p = v; }
 __device__ __forceinline__ void store_as(__half* p, float v) { *p = __float2half_rn(v); }
+__device__ __forceinline__ void store_as(__nv_bfloat16* p, float v) { *p = __float2bfloat16_rn(v); }
+
+// Gated feed-forward: up * act(gate), act = silu or relu (Activation in kernels.h). silu keeps the operation order
+// sigmoid = 1/(1+exp(-x)), x*sigmoid, up*silu.
+__device__ __forceinline__ float gated(int act, float gate, float up) {
+  if (act == 1) return __fmul_rn(up, fmaxf(gate, 0.f));
+  const float sig = __fdiv_rn(1.0f, 1.0f + expf(-gate));
+  return __fmul_rn(up, __fmul_rn(gate, sig));
+}
 
 }  // namespace nfai

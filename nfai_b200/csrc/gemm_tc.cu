@@ -18,6 +18,7 @@
 #include <cuda.h>
 
 #include "common.cuh"
+#include "gemm_epilogue.cuh"
 #include "gemm_tc.h"
 #include "kernels.h"
 
@@ -112,99 +113,6 @@ __device__ __forceinline__ void tmem_ld32(uint32_t taddr, float (&v)[32]) {
   asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
 #pragma unroll
   for (int i = 0; i < 32; ++i) v[i] = __uint_as_float(r[i]);
-}
-
-// ---- epilogues: two adjacent output columns (n, n+1) of row m; n is even -----------------------------------------
-// What the epilogue of a pair reads from memory: the residual pair of a plain store, the (cos, sin) of a rotated Q/K
-// pair. The callers fetch it for a whole block of pairs before they touch the accumulators: a loop of load -> add ->
-// store per pair runs at one memory round trip per pair (the store may alias the next load as far as the compiler
-// knows), which cost more than the tile's MMAs.
-// KIND >= 0 fixes the epilogue at compile time (the persistent kernel dispatches once per tile); -1 reads ep.kind.
-template <int KIND = -1>
-__device__ __forceinline__ float2 epilogue_aux(const GemmEpilogue& ep, uint32_t m, uint32_t n, uint32_t N) {
-  switch (KIND >= 0 ? KIND : (int)ep.kind) {
-    case GEMM_EPI_STORE: {
-      if (!ep.resid) break;
-      const float* res = ep.resid + (size_t)m * N;
-      if ((N & 1u) == 0) return __ldcg(reinterpret_cast<const float2*>(res + n));
-      return make_float2(__ldcg(res + n), n + 1 < N ? __ldcg(res + n + 1) : 0.f);
-    }
-    case GEMM_EPI_QKV_ROPE: {
-      if (n < ep.qDim + ep.kvDim) {
-        const uint32_t local = n < ep.qDim ? n : n - ep.qDim;
-        const uint32_t e = local % ep.d;
-        if (e < ep.ropeDim) return ep.rope_cs[(size_t)(ep.pos0 + m) * (ep.ropeDim / 2) + (e >> 1)];
-      }
-      break;
-    }
-    default: break;
-  }
-  return make_float2(0.f, 0.f);
-}
-
-template <int KIND = -1>
-__device__ __forceinline__ void epilogue_pair(const GemmEpilogue& ep, uint32_t m, uint32_t n, uint32_t N, float a, float b,
-                                              const float2 aux) {
-  switch (KIND >= 0 ? KIND : (int)ep.kind) {
-    case GEMM_EPI_STORE: {
-      float* out = ep.out_f32 + (size_t)m * N;
-      if ((N & 1u) == 0) {  // rows start on an 8-byte boundary: one store per pair
-        float2 r = make_float2(a, b);
-        if (ep.resid) {
-          r.x += aux.x;
-          r.y += aux.y;
-        }
-        *reinterpret_cast<float2*>(out + n) = r;
-      } else {
-        out[n] = ep.resid ? aux.x + a : a;
-        if (n + 1 < N) out[n + 1] = ep.resid ? aux.y + b : b;
-      }
-      break;
-    }
-    case GEMM_EPI_SILU_MUL: {  // columns (2j, 2j+1) = (gate_j, up_j); h_j = up * silu(gate), stored as float16
-      if (n + 1 < N) {
-        const float sig = __fdiv_rn(1.0f, 1.0f + expf(-a));
-        ep.out_f16[(size_t)m * (N / 2) + (n >> 1)] = __float2half_rn(__fmul_rn(b, __fmul_rn(a, sig)));
-      }
-      break;
-    }
-    case GEMM_EPI_QKV_ROPE: {  // columns [Q | K | V]; RoPE on adjacent pairs at position pos0 + m
-      const uint32_t pos = ep.pos0 + m;
-      if (n < ep.qDim + ep.kvDim) {
-        const uint32_t local = n < ep.qDim ? n : n - ep.qDim;
-        const uint32_t e = local % ep.d;
-        if (e < ep.ropeDim) {
-          const float2 cs = aux;
-          const float v1 = __fsub_rn(__fmul_rn(cs.x, a), __fmul_rn(cs.y, b));
-          const float v2 = __fadd_rn(__fmul_rn(cs.y, a), __fmul_rn(cs.x, b));
-          a = v1;
-          b = v2;
-        }
-        if (n < ep.qDim) {
-          // (n, local and the row lengths are even: pairs are naturally aligned)
-          *reinterpret_cast<float2*>(ep.out_f32 + (size_t)m * ep.qDim + n) = make_float2(a, b);
-        } else if (ep.kv_f16) {
-          __half* kc = reinterpret_cast<__half*>(ep.kcache) + (size_t)pos * ep.kvDim + local;
-          *reinterpret_cast<__half2*>(kc) = __floats2half2_rn(a, b);
-        } else {
-          float* kc = reinterpret_cast<float*>(ep.kcache) + (size_t)pos * ep.kvDim + local;
-          kc[0] = a;
-          kc[1] = b;
-        }
-      } else {
-        const uint32_t local = n - ep.qDim - ep.kvDim;
-        if (ep.kv_f16) {
-          __half* vc = reinterpret_cast<__half*>(ep.vcache) + (size_t)pos * ep.kvDim + local;
-          *reinterpret_cast<__half2*>(vc) = __floats2half2_rn(a, b);
-        } else {
-          float* vc = reinterpret_cast<float*>(ep.vcache) + (size_t)pos * ep.kvDim + local;
-          vc[0] = a;
-          vc[1] = b;
-        }
-      }
-      break;
-    }
-  }
 }
 
 // 32 consecutive output columns [n0, n0+32) of row m (n0 is a multiple of 32)
@@ -309,8 +217,8 @@ __global__ void __launch_bounds__(kGemmThreads) gemm_tc_kernel(const __grid_cons
     }
   } else if (warp == 1) {
     if (lane == 0) {
-      // instruction descriptor: D float32, A and B float16, both K-major, N = BN, M = 128
-      const uint32_t idesc = (1u << 4) | ((uint32_t)(BN >> 3) << 17) | ((uint32_t)(kBM >> 4) << 24);
+      // instruction descriptor: D float32, A and B of one 16-bit type (0 = float16, 1 = bfloat16), both K-major, N = BN, M = 128
+      const uint32_t idesc = (1u << 4) | (ep.operands_bf16 << 7) | (ep.operands_bf16 << 10) | ((uint32_t)(BN >> 3) << 17) | ((uint32_t)(kBM >> 4) << 24);
       for (uint32_t kt = 0; kt < KT; ++kt) {
         const uint32_t s = kt % STAGES;
         if (!bar_wait(full0 + 8 * s, (kt / STAGES) & 1)) { ok = false; break; }
@@ -444,7 +352,7 @@ __global__ void __launch_bounds__(kPThreadsGemm) gemm_tc_persistent_kernel(const
     }
   } else if (warp == 1) {
     if (lane == 0) {
-      const uint32_t idesc = (1u << 4) | ((uint32_t)(kPBN >> 3) << 17) | ((uint32_t)(kBM >> 4) << 24);
+      const uint32_t idesc = (1u << 4) | (ep.operands_bf16 << 7) | (ep.operands_bf16 << 10) | ((uint32_t)(kPBN >> 3) << 17) | ((uint32_t)(kBM >> 4) << 24);
       uint32_t it = 0, i = 0;
       for (uint32_t tile = blockIdx.x; tile < tiles && ok; tile += gridDim.x, ++i) {
         const uint32_t acc = i & 1;
@@ -479,7 +387,8 @@ __global__ void __launch_bounds__(kPThreadsGemm) gemm_tc_persistent_kernel(const
       // One instance per epilogue kind, chosen once per tile: the loops below are straight-line code for that kind.
       auto tile_epilogue = [&](auto kind_c) -> bool {
         constexpr int KIND = decltype(kind_c)::value;
-        constexpr bool kAux = KIND != GEMM_EPI_SILU_MUL;  // residual pairs / (cos, sin) pairs come from memory
+        // residual pairs / (cos, sin) pairs come from memory per row; a bias pair is the same for all rows of a lane's block
+        constexpr bool kAux = KIND == GEMM_EPI_STORE || KIND == GEMM_EPI_QKV_ROPE;
         float2 aux[16];
         // Q/K/V columns: everything that depends on the column only (which of Q, K, V; the position inside the head;
         // whether the pair is rotated) is the same for the 16 pairs of a lane in one block and is worked out once.
@@ -535,6 +444,11 @@ __global__ void __launch_bounds__(kPThreadsGemm) gemm_tc_persistent_kernel(const
             __syncwarp();
           }
           float2 cur[16];
+          float2 col_bias = make_float2(0.f, 0.f);
+          if constexpr (!kAux) {
+            const uint32_t n = n0 + c * 32 + col;
+            if (n < N) col_bias = epilogue_aux<KIND>(ep, 0, n, N);
+          }
           if constexpr (kAux) {
 #pragma unroll
             for (int rr = 0; rr < 16; ++rr) cur[rr] = aux[rr];
@@ -580,7 +494,7 @@ __global__ void __launch_bounds__(kPThreadsGemm) gemm_tc_persistent_kernel(const
               const uint32_t row = 2u * rr + (lane >> 4);
               const uint32_t m = m0 + lane_grp * 32 + row, n = n0 + c * 32 + col;
               if (m < M && n < N)
-                epilogue_pair<KIND>(ep, m, n, N, eb[row * 33 + col], eb[row * 33 + col + 1], kAux ? cur[rr] : make_float2(0.f, 0.f));
+                epilogue_pair<KIND>(ep, m, n, N, eb[row * 33 + col], eb[row * 33 + col + 1], kAux ? cur[rr] : col_bias);
             }
             __syncwarp();
           }
@@ -589,7 +503,8 @@ __global__ void __launch_bounds__(kPThreadsGemm) gemm_tc_persistent_kernel(const
       };
       switch (ep.kind) {
         case GEMM_EPI_STORE: ok = tile_epilogue(std::integral_constant<int, (int)GEMM_EPI_STORE>{}); break;
-        case GEMM_EPI_SILU_MUL: ok = tile_epilogue(std::integral_constant<int, (int)GEMM_EPI_SILU_MUL>{}); break;
+        case GEMM_EPI_GATED: ok = tile_epilogue(std::integral_constant<int, (int)GEMM_EPI_GATED>{}); break;
+        case GEMM_EPI_STORE_ACT: ok = tile_epilogue(std::integral_constant<int, (int)GEMM_EPI_STORE_ACT>{}); break;
         default: ok = tile_epilogue(std::integral_constant<int, (int)GEMM_EPI_QKV_ROPE>{}); break;
       }
       if (!ok) break;
@@ -757,7 +672,8 @@ uint32_t gemm_tc_splits(uint32_t M, uint32_t N, uint32_t K) {
 cudaError_t launch_gemm_tc(cudaStream_t s, const __half* A, const __half* W, uint32_t M, uint32_t N, uint32_t K,
                            const GemmEpilogue& ep, uint32_t* err) {
   if (!A || !W || !M || !N || !K || (K & 7u) || (((uintptr_t)A | (uintptr_t)W) & 15)) return cudaErrorInvalidValue;
-  if ((ep.kind == GEMM_EPI_SILU_MUL || ep.kind == GEMM_EPI_QKV_ROPE) && (N & 1u)) return cudaErrorInvalidValue;
+  if ((ep.kind == GEMM_EPI_GATED || ep.kind == GEMM_EPI_QKV_ROPE) && (N & 1u)) return cudaErrorInvalidValue;
+  if (ep.operands_bf16 > 1) return cudaErrorInvalidValue;
   // enough CTAs to pull weights with every SM when the chunk is a single row of tiles
   const uint32_t mtiles = (M + kBM - 1) / kBM;
   // enough 128 x 256 tiles to occupy most SMs: the persistent kernel (NFAI_GEMM_PERSISTENT=0 keeps the tile-per-CTA one)

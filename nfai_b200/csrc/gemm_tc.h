@@ -6,13 +6,17 @@
 
 namespace nfai {
 
-enum GemmEpilogueKind { GEMM_EPI_STORE = 0, GEMM_EPI_SILU_MUL = 1, GEMM_EPI_QKV_ROPE = 2 };
+enum GemmEpilogueKind { GEMM_EPI_STORE = 0, GEMM_EPI_GATED = 1, GEMM_EPI_QKV_ROPE = 2, GEMM_EPI_STORE_ACT = 3 };
 
 struct GemmEpilogue {
   int kind = GEMM_EPI_STORE;
   float* out_f32 = nullptr;      // STORE: [M][N]; QKV_ROPE: q rows [M][qDim]
   const float* resid = nullptr;  // STORE: optional [M][N] addend
-  __half* out_f16 = nullptr;     // SILU_MUL: [M][N/2]
+  const float* bias = nullptr;   // STORE, STORE_ACT, GATED: optional [N]
+  void* out_act = nullptr;       // GATED: [M][N/2], STORE_ACT: [M][N], of out_dtype
+  int out_dtype = 1;             // 0 float32, 1 float16, 2 bfloat16
+  int act = 0;                   // GATED: Activation (kernels.h)
+  uint32_t operands_bf16 = 0;    // 1: A and W are bfloat16 (both), 0: float16 (both)
   // QKV_ROPE
   void* kcache = nullptr;
   void* vcache = nullptr;
@@ -39,6 +43,10 @@ cudaError_t launch_gemm_tc(cudaStream_t s, const __half* A, const __half* W, uin
 // plain stream order (no programmatic dependent launch across the library's kernels).
 cudaError_t launch_rmsnorm_to_half(cudaStream_t s, const float* x, const float* gain, float eps, uint32_t M, uint32_t H,
                                    __half* out, bool after_collective = false);
+// The same product with any K and any alignment on the CUDA cores, A and W both of `dtype` (0 float32, 2 bfloat16): true
+// float32 models, and shapes the tensor-core kernel cannot take.
+cudaError_t launch_gemm_simt(cudaStream_t s, int dtype, const void* A, const void* W, uint32_t M, uint32_t N, uint32_t K,
+                             const GemmEpilogue& ep);
 // rows of the embedding matrix (float16) widened to float32: x[t] = E[tokens[t]].
 cudaError_t launch_embed_rows(cudaStream_t s, const __half* E, const uint32_t* tokens, uint32_t M, uint32_t H, float* x);
 cudaError_t launch_float_to_half(cudaStream_t s, const float* in, __half* out, size_t n);

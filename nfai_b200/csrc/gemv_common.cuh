@@ -144,6 +144,21 @@ __device__ __forceinline__ void load_x(const GemvParams& p, float* xs, float* re
     __syncthreads();
     return;
   }
+  if (!PERM && p.norm_groups > 1) {  // every part by its own root mean square; the scratch for them lies behind the gain
+    float* rms_of = xs + 2 * (size_t)K;
+    const uint32_t part = K / p.norm_groups;
+    __syncthreads();
+    for (uint32_t g = tid >> 5; g < p.norm_groups; g += kWarps) {
+      float sg = 0.f;
+      for (uint32_t i = tid & 31; i < part; i += 32) sg = fmaf(xs[g * part + i], xs[g * part + i], sg);
+      sg = warp_sum(sg);
+      if ((tid & 31) == 0) rms_of[g] = sqrtf(__fdiv_rn(sg, (float)part) + p.eps);
+    }
+    __syncthreads();
+    for (uint32_t i = tid; i < K; i += kThreads) xs[i] = __fmul_rn(__fdiv_rn(xs[i], rms_of[i / part]), gs[i]);
+    __syncthreads();
+    return;
+  }
   ss = warp_sum(ss);
   if ((tid & 31) == 0) red[tid >> 5] = ss;
   __syncthreads();
@@ -198,7 +213,7 @@ __device__ __forceinline__ void row_epilogue(const GemvParams& p, uint32_t row0,
 #pragma unroll
     for (int r = 0; r < R; ++r) {
       uint32_t n = row0 + r;
-      if (n < p.N) p.y[n] = p.resid ? __ldcg(p.resid + n) + acc[r] : acc[r];
+      if (n < p.N) p.y[n] = (p.resid ? __ldcg(p.resid + n) : 0.f) + (p.bias ? __ldg(p.bias + n) : 0.f) + acc[r];
     }
   } else if constexpr (EPI == EPI_QKV_ROPE) {
     static_assert(R % 2 == 0, "RoPE pairs adjacent rows");
@@ -237,16 +252,15 @@ __device__ __forceinline__ void row_epilogue(const GemvParams& p, uint32_t row0,
         store_as(vc + 1, b);
       }
     }
-  } else if constexpr (EPI == EPI_SILU_MUL) {
+  } else if constexpr (EPI == EPI_GATED) {
     static_assert(R % 2 == 0, "gate and up rows are interleaved");
 #pragma unroll
     for (int r = 0; r < R; r += 2) {
       uint32_t n = row0 + r;
       if (n >= p.N) break;
-      float gate = acc[r], up = acc[r + 1];
       // sigmoid = 1/(1+exp(-x)); silu = x*sigmoid; h = up*silu (SiLUShader.cs:121-123, ElementWiseMul A=up,B=silu)
-      float sig = __fdiv_rn(1.0f, 1.0f + expf(-gate));
-      p.y[n >> 1] = __fmul_rn(up, __fmul_rn(gate, sig));
+      const float gate = p.bias ? acc[r] + __ldg(p.bias + n) : acc[r], up = p.bias ? acc[r + 1] + __ldg(p.bias + n + 1) : acc[r + 1];
+      p.y[n >> 1] = gated(p.act, gate, up);
     }
   } else {  // EPI_LOGITS: store and keep the warp's best (lowest index among equal maxima)
 #pragma unroll
@@ -274,7 +288,14 @@ __device__ __forceinline__ void epi_preload(const GemvParams& p, uint32_t row0, 
 #pragma unroll
     for (int r = 0; r < R; ++r) {
       const uint32_t n = row0 + r < p.N ? row0 + r : p.N - 1;
-      pre[r] = p.resid ? __ldcg(p.resid + n) : 0.f;
+      pre[r] = (p.resid ? __ldcg(p.resid + n) : 0.f) + (p.bias ? __ldg(p.bias + n) : 0.f);
+    }
+  } else if constexpr (EPI == EPI_HYPER) {  // lane s holds stream s, lane 31 the bias
+    const uint32_t lane = threadIdx.x & 31;
+#pragma unroll
+    for (int r = 0; r < R; ++r) {
+      const uint32_t n = row0 + r < p.N ? row0 + r : p.N - 1;
+      pre[r] = lane < p.hyper.S ? __ldcg(p.hyper.x_in + (size_t)lane * p.N + n) : lane == 31 && p.bias ? __ldg(p.bias + n) : 0.f;
     }
   } else if constexpr (EPI == EPI_QKV_ROPE) {
 #pragma unroll
@@ -298,6 +319,31 @@ __device__ __forceinline__ void epi_preload(const GemvParams& p, uint32_t row0, 
 template <typename KVT, int R, int EPI>
 __device__ __forceinline__ void row_epilogue_pre(const GemvParams& p, uint32_t row0, const float (&acc)[R],
                                                  const float (&pre)[R], uint32_t pos, float& best_v, uint32_t& best_i) {
+  if constexpr (EPI == EPI_HYPER) {  // the whole warp: lane t makes stream t
+    const HyperWrite& h = p.hyper;
+    const uint32_t lane = threadIdx.x & 31;
+    const bool live = lane < h.S;
+    const float w_out = live ? __ldg(h.out + lane) : 0.f;
+    const float w_next = live ? (h.next_in ? __ldg(h.next_in + lane) : 1.f) : 0.f;
+    float v[R];
+#pragma unroll
+    for (int r = 0; r < R; ++r) v[r] = w_out * (acc[r] + __shfl_sync(0xffffffffu, pre[r], 31));
+    for (uint32_t s = 0; s < h.S; ++s) {
+      const float w = live ? __ldg(h.mix + s * h.S + lane) : 0.f;
+#pragma unroll
+      for (int r = 0; r < R; ++r) v[r] = fmaf(w, __shfl_sync(0xffffffffu, pre[r], s), v[r]);
+    }
+#pragma unroll
+    for (int r = 0; r < R; ++r) {
+      const uint32_t n = row0 + r;
+      const float u = warp_sum(w_next * v[r]);
+      if (n < p.N) {
+        if (live) h.x_out[(size_t)lane * p.N + n] = v[r];
+        if (lane == 0) h.u[n] = u;
+      }
+    }
+    return;
+  }
   if ((threadIdx.x & 31) != 0) return;
   if constexpr (EPI == EPI_STORE) {
     if (p.tp.push) {
@@ -307,7 +353,7 @@ __device__ __forceinline__ void row_epilogue_pre(const GemvParams& p, uint32_t r
 #pragma unroll
     for (int r = 0; r < R; ++r) {
       uint32_t n = row0 + r;
-      if (n < p.N) p.y[n] = p.resid ? pre[r] + acc[r] : acc[r];
+      if (n < p.N) p.y[(p.y_ring ? (size_t)(pos % p.y_ring) * p.y_stride : 0) + n] = pre[r] + acc[r];
     }
   } else if constexpr (EPI == EPI_QKV_ROPE) {
     static_assert(R % 2 == 0, "RoPE pairs adjacent rows");

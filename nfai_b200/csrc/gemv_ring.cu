@@ -324,7 +324,7 @@ cudaError_t launch_re(GemvEpilogue epi, int S, dim3 grid, size_t smem, cudaStrea
   switch (epi) {
     case EPI_STORE: return launch_x<WT, float, EPI_STORE>(S, grid, smem, s, pdl, p);
     case EPI_QKV_ROPE: return launch_x<WT, KVT, EPI_QKV_ROPE>(S, grid, smem, s, pdl, p);
-    case EPI_SILU_MUL: return launch_x<WT, float, EPI_SILU_MUL>(S, grid, smem, s, pdl, p);
+    case EPI_GATED: return launch_x<WT, float, EPI_GATED>(S, grid, smem, s, pdl, p);
     case EPI_LOGITS: return launch_x<WT, float, EPI_LOGITS>(S, grid, smem, s, pdl, p);
   }
   return cudaErrorInvalidValue;
@@ -347,7 +347,7 @@ uint32_t gemv_ring_grid(const GemvParams& p, int ctas_per_sm) {
 
 cudaError_t launch_gemv_ring(cudaStream_t s, int wdtype, int kvdtype, GemvEpilogue epi, const GemvParams& p, int S,
                              int ctas_per_sm, bool pdl) {
-  if ((epi == EPI_QKV_ROPE || epi == EPI_SILU_MUL) && (p.N % 2) != 0) return cudaErrorInvalidValue;
+  if ((epi == EPI_QKV_ROPE || epi == EPI_GATED) && (p.N % 2) != 0) return cudaErrorInvalidValue;
   const size_t smem = gemv_ring_smem(p, S);
   if (smem > 227 * 1024) return cudaErrorInvalidValue;
   dim3 grid(gemv_ring_grid(p, ctas_per_sm));

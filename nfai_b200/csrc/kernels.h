@@ -55,6 +55,8 @@ inline cudaError_t launch_pdl(void (*kernel)(KArgs...), dim3 grid, dim3 block, s
   cfg.numAttrs = 1;
   return cudaLaunchKernelEx(&cfg, kernel, static_cast<KArgs>(args)...);
 }
+// Integer environment switch; `dflt` when it is unset or empty.
+int env_int(const char* name, int dflt);
 // Prompt-path kernels overlap their launch and set-up with the predecessor's tail unless NFAI_PREFILL_PDL=0.
 bool prefill_pdl();
 
@@ -84,9 +86,27 @@ constexpr uint32_t kPrefetchChunk = 4096;
 enum GemvEpilogue {
   EPI_STORE = 0,     // y = acc (+ resid)
   EPI_QKV_ROPE = 1,  // rows are [Q | K | V]; RoPE on Q and K; K,V rows go to the cache at row pos
-  EPI_SILU_MUL = 2,  // rows are interleaved (gate_j, up_j); h_j = up_j * silu(gate_j)
-  EPI_LOGITS = 3     // y = acc and a per-CTA (max, lowest index) partial
+  EPI_GATED = 2,     // rows are interleaved (gate_j, up_j); h_j = up_j * act(gate_j)
+  EPI_LOGITS = 3,    // y = acc and a per-CTA (max, lowest index) partial
+  EPI_HYPER = 4      // y = acc is written into all residual streams (hyper-connections, see HyperWrite)
 };
+
+// Activation of a gated feed-forward.
+enum Activation { ACT_SILU = 0, ACT_RELU = 1 };
+
+// Hyper-connections: the residual is kept as S streams x_s. A sublayer reads u = sum_s in[s] x_s and its output y is
+// written back into all of them: x'_t = sum_s mix[s][t] x_s + out[t] y. The kernel that writes also forms what the NEXT
+// reader needs, u' = sum_t next_in[t] x'_t, so that the reader's prologue is the one of a plain residual.
+struct HyperWrite {
+  const float* x_in = nullptr;     // [S][N] streams before
+  float* x_out = nullptr;          // [S][N] streams after (may be x_in)
+  const float* mix = nullptr;      // [S][S], [from][to]
+  const float* out = nullptr;      // [S]
+  const float* next_in = nullptr;  // [S] weights of the next reader; null: the plain sum of the streams
+  float* u = nullptr;              // [N] what the next reader reads
+  uint32_t S = 0;                  // <= kMaxStreams
+};
+constexpr uint32_t kMaxStreams = 16;
 
 struct GemvParams {
   const void* W = nullptr;  // [N][K] row-major, float or half
@@ -95,7 +115,7 @@ struct GemvParams {
   const float* gain = nullptr;  // [K] RMSNorm gain, or null for no normalisation
   float eps = 0.f;
   const float* resid = nullptr;  // [N] or null
-  float* y = nullptr;            // [N] (EPI_STORE, EPI_LOGITS) or [N/2] (EPI_SILU_MUL)
+  float* y = nullptr;            // [N] (EPI_STORE, EPI_LOGITS) or [N/2] (EPI_GATED)
   // EPI_QKV_ROPE
   float* q_out = nullptr;
   void* kcache = nullptr;  // [ctx][kvDim] of the kv type
@@ -118,13 +138,19 @@ struct GemvParams {
   // (exchange tp.push_index)
   uint32_t v_lo = 0;
   uint32_t* tp_ticket = nullptr;
+  const float* bias = nullptr;  // [N] added to the row sums (EPI_STORE, EPI_GATED, EPI_HYPER)
+  int act = ACT_SILU;           // EPI_GATED
+  uint32_t norm_groups = 1;     // the prologue's RMS norm works on this many equal parts of x, each by its own mean
+  // EPI_STORE into a ring of rows: y is row (position % y_ring) of a buffer of rows y_stride floats apart (0 = plain y)
+  uint32_t y_ring = 0, y_stride = 0;
+  HyperWrite hyper;             // EPI_HYPER
 };
 
 // Tunable launch shape of the GEMV family.
 struct GemvTune {
   int mode = 0;           // 0 = register double-buffered streamer, 1 = per-warp shared-memory rings fed by bulk copies
                           // (stages of 2 rows x 2 KB)
-  int rows_per_warp = 2;  // mode 0: 1, 2 or 4 (EPI_QKV_ROPE and EPI_SILU_MUL need an even value); ring modes: always 2
+  int rows_per_warp = 2;  // mode 0: 1, 2 or 4 (EPI_QKV_ROPE and EPI_GATED need an even value); ring modes: always 2
   int unroll = 4;         // mode 0: 16-byte loads in flight per row per lane (2, 4 or 8); ring modes: stages per warp (1-4)
   int ctas_per_sm = 2;    // persistent grid = min(needed, 148 * ctas_per_sm) CTAs of 256 threads
   int split = 0;          // mode 0: warps sharing one row block (1, 2, 4, 8); 0 = chosen from the matrix shape
@@ -138,6 +164,8 @@ uint32_t gemv_ring_grid(const GemvParams& p, int ctas_per_sm);
 cudaError_t launch_gemv_ring(cudaStream_t s, int wdtype, int kvdtype, GemvEpilogue epi, const GemvParams& p, int S,
                              int ctas_per_sm, bool pdl);
 
+// wdtype: 0 = float32, 1 = float16, 2 = bfloat16 (bfloat16 and EPI_HYPER: register streamer only; EPI_QKV_ROPE is not
+// available for bfloat16 weights).
 // Number of CTAs the launch will use (the LM head needs it to size its partial buffers).
 uint32_t gemv_grid(int wdtype, GemvEpilogue epi, const GemvParams& p, const GemvTune& t);
 cudaError_t launch_gemv(cudaStream_t s, int wdtype, int kvdtype, GemvEpilogue epi, const GemvParams& p,

@@ -186,6 +186,11 @@ cudaError_t launch_ingest(cudaStream_t s, int src_dtype, int dst_dtype, const In
   else if (src_dtype == 0 && dst_dtype == 1) ingest_kernel<float, __half><<<grid, block, 0, s>>>(p);
   else if (src_dtype == 1 && dst_dtype == 0) ingest_kernel<__half, float><<<grid, block, 0, s>>>(p);
   else if (src_dtype == 1 && dst_dtype == 1) ingest_kernel<__half, __half><<<grid, block, 0, s>>>(p);
+  else if (src_dtype == 0 && dst_dtype == 2) ingest_kernel<float, __nv_bfloat16><<<grid, block, 0, s>>>(p);
+  else if (src_dtype == 1 && dst_dtype == 2) ingest_kernel<__half, __nv_bfloat16><<<grid, block, 0, s>>>(p);
+  else if (src_dtype == 2 && dst_dtype == 0) ingest_kernel<__nv_bfloat16, float><<<grid, block, 0, s>>>(p);
+  else if (src_dtype == 2 && dst_dtype == 1) ingest_kernel<__nv_bfloat16, __half><<<grid, block, 0, s>>>(p);
+  else if (src_dtype == 2 && dst_dtype == 2) ingest_kernel<__nv_bfloat16, __nv_bfloat16><<<grid, block, 0, s>>>(p);
   else return cudaErrorInvalidValue;
   return cudaGetLastError();
 }
