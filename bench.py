@@ -17,6 +17,10 @@ Prints ONE JSON line on rank 0.
              cannot run here) timed on the host cores on a few tokens of the same workload.
 
 --impl reference times that CPU port with all host threads on the same workload (rank 0 only).
+
+--design tometar is a workload of its own (one GPU, one JSON line): prompt and decode throughput of Tometar models whose
+layers have a real model's sizes (random weights), each beside a Llama model of the same width, depth, feed-forward and
+vocabulary, with the decode kernels of both timed alone.
 """
 import argparse
 import json
@@ -412,6 +416,138 @@ def run_ours(args, cfg):
         dist.destroy_process_group()
 
 
+# (width, layers, ff, latent attention, state space layer) of the Tometar workload and its Llama counterpart
+TOMETAR_SIZES = {
+    "1b": dict(width=2048, layers=16, ff=8192, vocab=128256,
+               latent=dict(heads=16, dim=128, rot_dim=64, vdim=128, kv_rank=512, window=1024),
+               ssm=dict(heads=64, vdim=64, state=128, groups=8, conv=4, norm_groups=8), llama=dict(qH=32, kvH=8, d=64)),
+    "3b": dict(width=3072, layers=28, ff=8192, vocab=128256,
+               latent=dict(heads=24, dim=128, rot_dim=64, vdim=128, kv_rank=512, window=2048),
+               ssm=dict(heads=96, vdim=64, state=128, groups=8, conv=4, norm_groups=8), llama=dict(qH=24, kvH=8, d=128)),
+}
+
+
+def tometar_config(z):
+    """Latent attention and state space layers in turn, all with a feed-forward."""
+    la = dict(z["latent"])
+    window = la.pop("window")
+    la.update(mask={"size": window}, rot={"base": 500000.0, "dims": la["rot_dim"]}, scale=(la["dim"] + la["rot_dim"]) ** -0.5)
+    layers = [{"type": "latent_attention", "mixer": la, "mlp": {"kind": "dense", "ff": z["ff"]}} if i % 2 == 0 else
+              {"type": "mamba2", "mixer": z["ssm"], "mlp": {"kind": "dense", "ff": z["ff"]}} for i in range(z["layers"])]
+    return {"architecture": "Tometar", "layers": layers, "norm": {"eps": 1e-5}, "streams": 4, "vocab": z["vocab"], "width": z["width"]}
+
+
+def tometar_tensors(cfg, seed):
+    """Random bfloat16 weights; large tensors repeat one block of normal draws from different places."""
+    import numpy as np
+
+    from nfai_b200 import _lib, config_tensors
+    rng = np.random.default_rng(seed)
+    block = rng.standard_normal((1 << 23) + 1).astype(np.float32)
+
+    def bits(a):
+        return (np.ascontiguousarray(a, np.float32).view(np.uint32) >> 16).astype(np.uint16)
+    for name, shape in config_tensors(cfg).items():
+        n = int(np.prod(shape))
+        last = name.split(".")[-1]
+        if last.startswith("norm"):
+            v = np.ones(n, np.float32)
+        elif ".hc" in name:
+            v = np.eye(shape[0], dtype=np.float32).ravel() if last == "mix" else np.full(n, 1.0 / shape[0] if last == "in" else 1.0, np.float32)
+        elif last == "A_log":
+            v = np.linspace(0.0, 2.7, n, dtype=np.float32)
+        elif last == "dt_bias":
+            v = np.full(n, -4.0, np.float32)
+        elif last == "conv":
+            v = block[:n] * 0.5
+        else:
+            k = rng.integers(0, block.size // 2)
+            v = np.resize(block[k:], n) * (0.02 if len(shape) > 1 else 0.01)
+        yield name, bits(v).reshape(shape), _lib.BF16
+
+
+def run_tometar(args):
+    import numpy as np
+    import torch
+
+    from nfai_b200 import LlamaModel, LlamaModelFactory, PlannedModel, synth, synthetic_tensors
+    T, K = args.design_prompt, args.steps
+    peak, peak_kind = measured_peak()
+    sus, burst, _ = measured_tflops()
+    factory = LlamaModelFactory(0)
+    sampler = ClockSampler(0)
+    sampler.start()
+
+    def measure(model, reset):
+        """Prompt of T tokens (median of 5, host clock with a synchronise on both sides), then K decode steps behind it."""
+        prompt = np.random.default_rng(args.seed).integers(0, model.V, T)
+        times = []
+        for i in range(8):
+            reset()
+            torch.cuda.synchronize()
+            t0 = time.perf_counter()
+            _, tk = model.prefill(prompt, want_logits=False)
+            torch.cuda.synchronize()
+            if i >= 3:
+                times.append(time.perf_counter() - t0)
+        snap = model.snapshot()
+        model.decode_greedy(tk, max(3, args.warmup))
+        ms = []
+        for _ in range(5):
+            snap.restore()
+            ms.append(model.decode_greedy(tk, K)[1] / K)
+        snap.restore()
+        t0 = time.perf_counter()
+        x = tk
+        for _ in range(K):
+            _, x = model.decode(x, want_logits=False)
+        e2e = (time.perf_counter() - t0) / K
+        snap.restore()
+        kern = {}
+        for name in model.KERNELS:
+            kms, kb = model.profile_kernel(name, 32 if name != "lm_head" else 8)
+            kern[name] = {"us": kms * 1e3, "gbs": kb / (kms * 1e-3) / 1e9, "frac_of_copy_peak": kb / (kms * 1e-3) / 1e9 / peak}
+        snap.close()
+        pf, step = statistics.median(times), statistics.median(ms)
+        return {"prefill_tokens": T, "prefill_ms": pf * 1e3, "prefill_tok_s": T / pf, "decode_ms": step, "decode_tok_s": 1e3 / step,
+                "decode_e2e_tok_s": 1 / e2e, "launches_per_step": model.step_launches(), "kernels": kern}
+
+    out = {}
+    for size in args.sizes.split(","):
+        z = TOMETAR_SIZES[size]
+        cfg = tometar_config(z)
+        m = PlannedModel.from_tensors(factory.ctx, cfg, tometar_tensors(cfg, args.seed), T + K + 64, "bf16")
+        ours = measure(m, m.reset)
+        m.Dispose()
+        la, sm, H, n = z["latent"], z["ssm"], z["width"], z["layers"]
+        p_la = (H * (la["heads"] * (la["dim"] + la["rot_dim"] + 2 * la["vdim"]) + la["kv_rank"] + la["rot_dim"])
+                + la["heads"] * (la["dim"] + la["vdim"]) * la["kv_rank"])
+        inner = sm["heads"] * sm["vdim"]
+        p_ss = H * (3 * inner + 2 * sm["groups"] * sm["state"] + sm["heads"])
+        params = n // 2 * (p_la + p_ss) + n * 3 * H * z["ff"]
+        ours["layer_matrix_params"] = params
+        ours["weight_gb_per_step"] = 2 * (params + z["vocab"] * H) / 1e9
+        ours["step_frac_of_copy_peak"] = ours["weight_gb_per_step"] / (ours["decode_ms"] * 1e-3) / peak
+        ours["prefill_matrix_tflops"] = 2.0 * params * T / (ours["prefill_ms"] * 1e-3) / 1e12
+        ours["prefill_frac_of_sustained_bf16"] = ours["prefill_matrix_tflops"] / sus
+        lc = synth.ModelConfig(f"llama-{size}", H, n, z["llama"]["qH"], z["llama"]["kvH"], z["llama"]["d"], z["ff"], z["vocab"], "f16")
+        lm = LlamaModel(factory.ctx, synth.metadata(lc), synthetic_tensors(lc, args.seed), T + K + 64)
+        like = measure(lm, lm.reset)
+        lm.Dispose()
+        lp = lc.streamed_matrix_params() - lc.V * lc.H
+        like["layer_matrix_params"] = lp
+        like["weight_gb_per_step"] = 2 * (lp + lc.V * lc.H) / 1e9
+        like["step_frac_of_copy_peak"] = like["weight_gb_per_step"] / (like["decode_ms"] * 1e-3) / peak
+        like["prefill_matrix_tflops"] = 2.0 * lp * T / (like["prefill_ms"] * 1e-3) / 1e12
+        like["prefill_frac_of_sustained_bf16"] = like["prefill_matrix_tflops"] / sus
+        out[size] = {"config": z, "tometar": ours, "llama": like}
+    factory.Dispose()
+    print(json.dumps({"metric": "Tometar prompt and decode throughput (batch 1)", "unit": "tok/s", "n_gpus": 1, "steps": K, "data": "synthetic",
+                      "dtype": "bf16 weights and operands, f32 residual, norms, scores and state; Llama: f16", "peak_hbm_gbs": peak,
+                      "peak_kind": peak_kind, "peak_bf16_tflops_sustained": sus, "sizes": out, "clocks": sampler.stop(),
+                      "l2": "every step streams all weights (larger than L2)"}), flush=True)
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -428,7 +564,13 @@ def main():
     ap.add_argument("--nccl-allreduce", action="store_true", help="N > 1: use NCCL all-reduces instead of the peer-memory kernel")
     ap.add_argument("--prompt-len", type=int, default=0,
                     help="0 = the configuration's own prompt length (c1 128, c2 2048, c3 1024, c4 32768)")
+    ap.add_argument("--design", default="llama", choices=["llama", "tometar"], help="tometar: the workload described above")
+    ap.add_argument("--sizes", default="1b,3b", help="--design tometar: which of its sizes")
+    ap.add_argument("--design-prompt", type=int, default=2048, help="--design tometar: prompt length")
     args = ap.parse_args()
+    if args.design == "tometar":
+        run_tometar(args)
+        return
     global PROMPT_LEN, MIN_TIMED_S
     MIN_TIMED_S = args.min_timed_s
     PROMPT_LEN = args.prompt_len or {"c2": 2048, "c3": 1024, "c4": 32768}.get(args.config, 128)

@@ -369,6 +369,10 @@ int nfai_op_attn_decode_static(nfai_ctx* ctx, const float* q, const void* kcache
  *           the reference never dispatches with more than one row. */
 int nfai_op_gemm_f16(nfai_ctx* ctx, const void* A, const void* W, uint32_t M, uint32_t N, uint32_t K, float* C);
 
+/* The same product for any operand type: dtype NFAI_F16 or NFAI_BF16 on the tensor cores (K % 8 == 0, 16-byte aligned; other
+ * shapes of NFAI_BF16 on the CUDA cores), NFAI_F32 in true float32 on the CUDA cores. No counterpart in the reference. */
+int nfai_op_gemm(nfai_ctx* ctx, const void* A, const void* W, int dtype, uint32_t M, uint32_t N, uint32_t K, float* C);
+
 /* logits = W * RMSNorm(x) (W[V][H]) and the lowest index of their maximum into *argmax_out (device).
  * replaces: output RMSNorm + LM-head MatrixMultiplyShader (LlamaModel.cs:58-67,160-163) and
  *           SamplingUtils.ArgMax (SamplingUtils.cs:55-56). */

@@ -1591,7 +1591,7 @@ int nfai_op_gemv(nfai_ctx* c, const void* W, int dtype, uint32_t N, uint32_t K, 
                  const float* resid, float* y) {
   int rc = op_begin(c);
   if (rc) return rc;
-  if (!W || !x || !y || bad_dtype(dtype) || !N || !K) return fail(c, NFAI_ERR_ARG, "bad argument");
+  if (!W || !x || !y || (bad_dtype(dtype) && dtype != NFAI_BF16) || !N || !K) return fail(c, NFAI_ERR_ARG, "bad argument");
   GemvParams p;
   p.W = W; p.N = N; p.K = K; p.x = x; p.gain = gain; p.eps = eps; p.resid = resid; p.y = y;
   GemvTune t;
@@ -1663,13 +1663,25 @@ int nfai_op_attn_decode(nfai_ctx* c, const float* q, const void* kcache, const v
 int nfai_op_gemm_f16(nfai_ctx* c, const void* A, const void* W, uint32_t M, uint32_t N, uint32_t K, float* C) {
   int rc = op_begin(c);
   if (rc) return rc;
-  if (!A || !W || !C || !M || !N || !K) return fail(c, NFAI_ERR_ARG, "bad argument");
   if (K % 8) return fail(c, NFAI_ERR_ARG, "K must be a multiple of 8");
   if (((uintptr_t)A | (uintptr_t)W) & 15) return fail(c, NFAI_ERR_ARG, "A and W must be 16-byte aligned");
-  CU(c, cudaMemsetAsync(c->dev_err, 0, 4, c->stream));
+  return nfai_op_gemm(c, A, W, NFAI_F16, M, N, K, C);
+}
+
+int nfai_op_gemm(nfai_ctx* c, const void* A, const void* W, int dtype, uint32_t M, uint32_t N, uint32_t K, float* C) {
+  int rc = op_begin(c);
+  if (rc) return rc;
+  if (!A || !W || !C || !M || !N || !K || (bad_dtype(dtype) && dtype != NFAI_BF16)) return fail(c, NFAI_ERR_ARG, "bad argument");
   GemmEpilogue ep;
   ep.kind = GEMM_EPI_STORE;
   ep.out_f32 = C;
+  const bool tc = dtype != NFAI_F32 && K % 8 == 0 && (((uintptr_t)A | (uintptr_t)W) & 15) == 0;
+  if (!tc) {
+    if (dtype == NFAI_F16) return fail(c, NFAI_ERR_ARG, "float16 operands need K % 8 == 0 and 16-byte alignment");
+    return op_end(c, launch_gemm_simt(c->stream, dtype, A, W, M, N, K, ep));
+  }
+  ep.operands_bf16 = dtype == NFAI_BF16;
+  CU(c, cudaMemsetAsync(c->dev_err, 0, 4, c->stream));
   const uint32_t Z = env_int("NFAI_GEMM_SPLIT", 1) ? gemm_tc_splits(M, N, K) : 1;
   if (Z > 1) {
     ep.scratch_floats = (size_t)Z * M * N;

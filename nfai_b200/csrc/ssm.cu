@@ -11,6 +11,10 @@
 
 namespace nfai {
 
+// ssm_chunk.cu
+bool ssm_chunk_supported(const SsmSpec& s);
+cudaError_t launch_ssm_chunked(cudaStream_t s, const SsmParams& p, uint32_t T);
+
 namespace {
 
 constexpr int kStepV = 32;  // state rows (values of one head) per CTA
@@ -266,8 +270,6 @@ cudaError_t launch_ssm_step(cudaStream_t s, const SsmParams& p, bool pdl) {
   return launch_pdl(kern, dim3(p.spec.heads, (p.spec.vdim + kStepV - 1) / kStepV), dim3(256), smem, s, pdl, p);
 }
 
-size_t ssm_chunk_floats(const SsmSpec& s, uint32_t T) { (void)s; (void)T; return 0; }
-
 cudaError_t launch_ssm_prefill(cudaStream_t s, const SsmParams& p, uint32_t T) {
   if (!T) return cudaErrorInvalidValue;
   const dim3 cgrid((p.spec.channels() + p.spec.heads + 255) / 256, (T + 7) / 8);
@@ -277,6 +279,9 @@ cudaError_t launch_ssm_prefill(cudaStream_t s, const SsmParams& p, uint32_t T) {
   const uint32_t n = T < p.spec.taps ? T : p.spec.taps;
   e = launch_pdl(ssm_ring_kernel, dim3((p.spec.in_rows() + 255) / 256, n), dim3(256), 0, s, prefill_pdl(), p, T);
   if (e != cudaSuccess) return e;
+  // portions long enough to fill the tensor cores' tiles: chunk by chunk (NFAI_SSM_CHUNK=0 keeps the token-by-token scan)
+  static const bool chunked = env_int("NFAI_SSM_CHUNK", 1) != 0;
+  if (p.xbc_dtype == 2 && chunked && T >= 32 && p.chunk && ssm_chunk_supported(p.spec)) return launch_ssm_chunked(s, p, T);
   return p.xbc_dtype == 2 ? launch_scan<__nv_bfloat16>(s, p, T) : launch_scan<float>(s, p, T);
 }
 

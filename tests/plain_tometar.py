@@ -3,12 +3,19 @@
 Used only by the tests; shares no code with the library. A sequence is evaluated token by token with everything that
 earlier tokens left behind kept in a `State`, so prompts, portions and decoding are the same computation here.
 Weights are a dict name -> float array (linear weights [out, in]).
+
+`act` and `cache` (identity by default) are applied where a 16-bit model rounds: `act` to the operands of matrix products and
+to what a convolution hands on, `cache` to the rows an attention layer keeps.
 """
 import json
 import os
 import struct
 
 import numpy as np
+
+
+def same(v):
+    return v
 
 
 # ---- mechanisms ---------------------------------------------------------------------------------------------------
@@ -54,25 +61,25 @@ def hyper_write(streams, y, w_mix, w_out):
     return w_mix.T @ streams + np.outer(w_out, y)
 
 
-def latent_attention(h, W, pre, spec, eps, pos, past):
+def latent_attention(h, W, pre, spec, eps, pos, past, act=same, cache=same):
     """`past` holds (latent, rotated key) of every earlier position; this position's pair is appended."""
     H, d, r, dv, R = spec["heads"], spec["dim"], spec["rot_dim"], spec["vdim"], spec["kv_rank"]
     base, dims = spec["rot"]["base"], spec["rot"]["dims"]
     q = (W[pre + "q"] @ h).reshape(H, d + r)
-    qu, qr = q[:, :d], rotate_half(q[:, d:], pos, base, dims)
+    qu, qr = act(q[:, :d]), act(rotate_half(q[:, d:], pos, base, dims))
     kv = W[pre + "dkv"] @ h
-    past.append((rms_norm(kv[:R], W[pre + "dkv.norm"], eps), rotate_half(kv[R:], pos, base, dims)))
+    past.append((cache(rms_norm(kv[:R], W[pre + "dkv.norm"], eps)), cache(rotate_half(kv[R:], pos, base, dims))))
     lo = max(0, pos - spec["mask"]["size"] + 1)
     C = np.stack([c for c, _ in past[lo:]])
     Kr = np.stack([k for _, k in past[lo:]])
-    Ku = (C @ W[pre + "uk"].T).reshape(-1, H, d)
-    V = (C @ W[pre + "uv"].T).reshape(-1, H, dv)
+    Ku = act(C @ W[pre + "uk"].T).reshape(-1, H, d)
+    V = act(C @ W[pre + "uv"].T).reshape(-1, H, dv)
     out = np.empty((H, dv))
     for i in range(H):
         s = (Ku[:, i] @ qu[i] + Kr @ qr[i]) * spec["scale"]
         out[i] = softmax(s) @ V[:, i]
     o = out.reshape(-1) * sigmoid(W[pre + "g"] @ h)
-    return W[pre + "o"] @ o
+    return W[pre + "o"] @ act(o)
 
 
 def short_conv(history, w, b):
@@ -104,25 +111,25 @@ def grouped_norm(y, w, parts, eps):
     return g.reshape(-1) * w
 
 
-def mamba2(h, W, pre, spec, eps, st):
+def mamba2(h, W, pre, spec, eps, st, act=same):
     heads, V, N, G = spec["heads"], spec["vdim"], spec["state"], spec["groups"]
     inner = heads * V
     u = W[pre + "in"] @ h
     z, xbc, dt = u[:inner], u[inner:2 * inner + 2 * G * N], u[2 * inner + 2 * G * N:]
     st["conv"].append(xbc)
-    c = short_conv(st["conv"], W[pre + "conv"], W[pre + "conv.b"])
+    c = act(short_conv(st["conv"], W[pre + "conv"], W[pre + "conv.b"]))
     st["conv"] = st["conv"][-W[pre + "conv"].shape[1]:]
     x, B, C = c[:inner].reshape(heads, V), c[inner:inner + G * N].reshape(G, N), c[inner + G * N:].reshape(G, N)
     dt = softplus(dt + W[pre + "dt_bias"])
     st["S"], y = ssm_step(st["S"], x, B, C, dt, W[pre + "A_log"], W[pre + "D"], G)
     y = grouped_norm(y.reshape(-1) * silu(z), W[pre + "norm"], spec["norm_groups"], eps)
-    return W[pre + "o"] @ y
+    return W[pre + "o"] @ act(y)
 
 
-def feed_forward(h, W, pre):
+def feed_forward(h, W, pre, act=same):
     gate = W[pre + "gate"] @ h + W[pre + "gate.b"]
     up = W[pre + "up"] @ h + W[pre + "up.b"]
-    return W[pre + "down"] @ (np.maximum(gate, 0.0) * up) + W[pre + "down.b"]
+    return W[pre + "down"] @ act(np.maximum(gate, 0.0) * up) + W[pre + "down.b"]
 
 
 # ---- the model ----------------------------------------------------------------------------------------------------
@@ -138,34 +145,34 @@ class State:
                 self.layers.append({"S": np.zeros((m["heads"], m["state"], m["vdim"])), "conv": []})
 
 
-def step(cfg, W, st, token, taps=None):
+def step(cfg, W, st, token, taps=None, act=same, cache=same):
     """Logits of one token; `taps` (a list) receives the sum of the streams after every layer."""
     eps, n = cfg["norm"]["eps"], cfg["streams"]
     X = np.tile(W["embed"][int(token)].astype(np.float64), (n, 1))
     for i, L in enumerate(cfg["layers"]):
         p = f"l{i}."
-        h = rms_norm(hyper_read(X, W[p + "hc1.in"]), W[p + "norm1"], eps)
+        h = act(rms_norm(hyper_read(X, W[p + "hc1.in"]), W[p + "norm1"], eps))
         if L["type"] == "latent_attention":
-            y = latent_attention(h, W, p + "mix.", L["mixer"], eps, st.pos, st.layers[i])
+            y = latent_attention(h, W, p + "mix.", L["mixer"], eps, st.pos, st.layers[i], act, cache)
         else:
-            y = mamba2(h, W, p + "mix.", L["mixer"], eps, st.layers[i])
+            y = mamba2(h, W, p + "mix.", L["mixer"], eps, st.layers[i], act)
         X = hyper_write(X, y, W[p + "hc1.mix"], W[p + "hc1.out"])
         if L["mlp"] is not None:
-            h = rms_norm(hyper_read(X, W[p + "hc2.in"]), W[p + "norm2"], eps)
-            X = hyper_write(X, feed_forward(h, W, p + "mlp."), W[p + "hc2.mix"], W[p + "hc2.out"])
+            h = act(rms_norm(hyper_read(X, W[p + "hc2.in"]), W[p + "norm2"], eps))
+            X = hyper_write(X, feed_forward(h, W, p + "mlp.", act), W[p + "hc2.mix"], W[p + "hc2.out"])
         if taps is not None:
             taps.append(X.sum(0))
     st.pos += 1
-    return W["head"] @ rms_norm(X.sum(0), W["final.norm"], eps)
+    return W["head"] @ act(rms_norm(X.sum(0), W["final.norm"], eps))
 
 
-def forward(cfg, W, tokens, st=None, taps=None):
+def forward(cfg, W, tokens, st=None, taps=None, act=same, cache=same):
     """[len(tokens), vocab] logits; `taps` receives one list of layer outputs per token."""
     st = st or State(cfg)
     out = []
     for t in tokens:
         tp = [] if taps is not None else None
-        out.append(step(cfg, W, st, t, tp))
+        out.append(step(cfg, W, st, t, tp, act, cache))
         if taps is not None:
             taps.append(tp)
     return np.array(out)
