@@ -131,7 +131,7 @@ cudaError_t launch_gemv(cudaStream_t s, int wdtype, int kvdtype, GemvEpilogue ep
   dim3 grid(gemv_grid(wdtype, epi, p, t));
   p.split_log2 = gemv_split_log2(wdtype, vec, R, p, t);
   if (p.norm_groups > 1 && (!p.gain || p.K % p.norm_groups)) return cudaErrorInvalidValue;
-  size_t smem = (kSmemHeader + (size_t)p.K * (p.gain ? 2 : 1) + (p.norm_groups > 1 ? p.norm_groups : 0)) * sizeof(float);
+  size_t smem = (kSmemHeader + (size_t)p.K * (p.gain ? 2 : 1)) * sizeof(float);
   if (smem > 227 * 1024) return cudaErrorInvalidValue;
   if (wdtype == 2 || epi == EPI_HYPER) {
     if (epi == EPI_QKV_ROPE || (epi == EPI_HYPER && (!p.hyper.S || p.hyper.S > kMaxStreams))) return cudaErrorInvalidValue;

@@ -144,18 +144,19 @@ __device__ __forceinline__ void load_x(const GemvParams& p, float* xs, float* re
     __syncthreads();
     return;
   }
-  if (!PERM && p.norm_groups > 1) {  // every part by its own root mean square; the scratch for them lies behind the gain
-    float* rms_of = xs + 2 * (size_t)K;
+  if (!PERM && p.norm_groups > 1) {  // every part by its own root mean square: a warp sums and scales whole parts
     const uint32_t part = K / p.norm_groups;
     __syncthreads();
     for (uint32_t g = tid >> 5; g < p.norm_groups; g += kWarps) {
+      float* xg = xs + g * part;
+      const float* gg = gs + g * part;
       float sg = 0.f;
-      for (uint32_t i = tid & 31; i < part; i += 32) sg = fmaf(xs[g * part + i], xs[g * part + i], sg);
-      sg = warp_sum(sg);
-      if ((tid & 31) == 0) rms_of[g] = sqrtf(__fdiv_rn(sg, (float)part) + p.eps);
+#pragma unroll 4
+      for (uint32_t i = tid & 31; i < part; i += 32) sg = fmaf(xg[i], xg[i], sg);
+      const float rms_g = sqrtf(__fdiv_rn(warp_sum(sg), (float)part) + p.eps);
+#pragma unroll 4
+      for (uint32_t i = tid & 31; i < part; i += 32) xg[i] = __fmul_rn(__fdiv_rn(xg[i], rms_g), gg[i]);
     }
-    __syncthreads();
-    for (uint32_t i = tid; i < K; i += kThreads) xs[i] = __fmul_rn(__fdiv_rn(xs[i], rms_of[i / part]), gs[i]);
     __syncthreads();
     return;
   }

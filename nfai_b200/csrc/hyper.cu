@@ -43,7 +43,7 @@ __device__ __forceinline__ void stv(float* p, const Vec<V>& v) {
 
 // ST >= S streams held in registers; V elements per thread and step
 template <int ST, int V>
-__global__ void __launch_bounds__(256) hyper_rows_kernel(const HyperRows p) {
+__global__ void __launch_bounds__(256, ST <= 4 ? 3 : 1) hyper_rows_kernel(const HyperRows p) {
   extern __shared__ __align__(16) float hsm[];
   float* us = hsm;  // [H] combined row
   __shared__ float w_mix[kMaxStreams * kMaxStreams], w_out[kMaxStreams], w_in[kMaxStreams], red[8];
@@ -61,6 +61,7 @@ __global__ void __launch_bounds__(256) hyper_rows_kernel(const HyperRows p) {
   float* Xo = p.X_out ? p.X_out + (size_t)blockIdx.x * S * H : nullptr;
   const size_t erow = p.tokens ? (size_t)p.tokens[blockIdx.x] * H : 0;
   float ss = 0.f;
+#pragma unroll 1
   for (uint32_t i = tid * V; i < H; i += 256 * V) {
     Vec<V> x[ST];
     if (p.tokens) {
@@ -137,9 +138,10 @@ template <int ST>
 cudaError_t launch_st(cudaStream_t s, const HyperRows& p, uint32_t n) {
   const size_t smem = (size_t)p.H * 4;
   if (smem > 200 * 1024) return cudaErrorInvalidValue;
-  auto k4 = hyper_rows_kernel<ST, 4>;
-  auto k1 = hyper_rows_kernel<ST, 1>;
-  auto kern = p.H % 4 == 0 ? k4 : k1;
+  auto kern = hyper_rows_kernel<ST, 1>;
+  if constexpr (ST <= 8) {  // more streams would not fit the register file in quads
+    if (p.H % 4 == 0) kern = hyper_rows_kernel<ST, 4>;
+  }
   if (smem > 40 * 1024) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return e;

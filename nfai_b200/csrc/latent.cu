@@ -465,10 +465,26 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const LatentParams p) 
   for (uint32_t i = threadIdx.x; i < rank; i += 256) store_as(c + i, __fmul_rn(__fdiv_rn(kv[i], rms), p.lat_gain[i]));
   CT* k = reinterpret_cast<CT*>(p.kr_cache) + (size_t)pos * rot;
   for (uint32_t i = threadIdx.x; i < rot; i += 256) store_as(k + i, rotated(kv + rank, i, s.rope_dims, cs));
-  CT* q = reinterpret_cast<CT*>(p.q) + (size_t)t * s.q_rows();
-  for (uint32_t i = threadIdx.x; i < s.q_rows(); i += 256) {
-    const uint32_t h = i / hd, e = i - h * hd;
-    store_as(q + i, e < s.dim ? row[i] : rotated(row + (size_t)h * hd + s.dim, e - s.dim, s.rope_dims, cs));
+  // a warp per head: four values a lane where the layout allows it
+  const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const bool quads = s.dim % 4 == 0 && hd % 4 == 0 && p.in_ld % 4 == 0;
+  for (uint32_t h = warp; h < s.heads; h += 8) {
+    const float* src = row + (size_t)h * hd;
+    CT* q = reinterpret_cast<CT*>(p.q) + (size_t)t * s.q_rows() + (size_t)h * hd;
+    if (quads) {
+      for (uint32_t i = lane * 4; i < s.dim; i += 128) {
+        const float4 v = *reinterpret_cast<const float4*>(src + i);
+        if constexpr (sizeof(CT) == 2) {
+          __nv_bfloat162 o[2] = {__floats2bfloat162_rn(v.x, v.y), __floats2bfloat162_rn(v.z, v.w)};
+          *reinterpret_cast<uint2*>(q + i) = *reinterpret_cast<uint2*>(o);
+        } else {
+          *reinterpret_cast<float4*>(q + i) = v;
+        }
+      }
+    } else {
+      for (uint32_t i = lane; i < s.dim; i += 32) store_as(q + i, src[i]);
+    }
+    for (uint32_t i = lane; i < rot; i += 32) store_as(q + s.dim + i, rotated(src + s.dim, i, s.rope_dims, cs));
   }
 }
 

@@ -1,5 +1,5 @@
 // Windowed causal attention of a prompt portion over expanded latents on the warp-level tensor cores (bfloat16 operands,
-// float32 accumulators). A CTA owns 64 tokens of one head (4 warps x 16 rows) and walks only the key tiles its tokens'
+// float32 accumulators). A CTA owns 16 tokens per warp of one head and walks only the key tiles its tokens'
 // windows reach. A key row is the head's unrotated part beside the rotated part all heads share; the two are brought
 // together in shared memory. Scores, running maximum, exponentials and sums are float32; the weights go into the second
 // product as a bfloat16 head and remainder (two MMAs, relative error ~2^-17), so that they keep more than the operand type.
@@ -11,7 +11,6 @@ namespace nfai {
 
 namespace {
 
-constexpr int kM = 64, kN = 64, kThr = 128;
 
 __device__ __forceinline__ uint32_t pack_bf(float a, float b) {
   __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
@@ -40,10 +39,12 @@ __device__ __forceinline__ float ex2(float x) {
   return y;
 }
 
-template <int DV>
-__global__ void __launch_bounds__(kThr) latent_prefill_mma_kernel(const LatentParams p, const uint32_t T, const uint32_t DQ,
+// W warps of 16 tokens, key tiles of kN positions
+template <int DV, int W, int kN>
+__global__ void __launch_bounds__(W * 32, DV <= 128 ? 2 : 1) latent_prefill_mma_kernel(const LatentParams p, const uint32_t T, const uint32_t DQ,
                                                                   const int vec) {
   // DQ: dim + rot rounded up to 16
+  constexpr int kM = W * 16, kThr = W * 32;
   extern __shared__ __align__(16) unsigned char lp_smem[];
   const LatentSpec& s = p.spec;
   const uint32_t dim = s.dim, rot = s.rot, hd = dim + rot, vdim = s.vdim;
@@ -241,25 +242,31 @@ __global__ void __launch_bounds__(kThr) latent_prefill_mma_kernel(const LatentPa
   }
 }
 
-size_t mma_smem(uint32_t DQ, uint32_t DV) { return ((size_t)(kM + 2 * kN) * (DQ + 8) + (size_t)2 * kN * (DV + 8)) * 2; }
+size_t mma_smem(uint32_t DQ, uint32_t DV, uint32_t kM, uint32_t kN) { return ((size_t)(kM + 2 * kN) * (DQ + 8) + (size_t)2 * kN * (DV + 8)) * 2; }
 uint32_t value_width(uint32_t vdim) { return vdim <= 32 ? 32 : vdim <= 64 ? 64 : vdim <= 128 ? 128 : vdim <= 256 ? 256 : 0; }
+
+// 8 warps and tiles of 32 positions: two CTAs per SM share the tensor cores, and 128 tokens share a tile (measured against
+// 4 and 8 warps with 32 and 64 positions).
+constexpr int kWarpsPerCta = 8, kTilePositions = 32;
 
 template <int DV>
 cudaError_t launch_dv(cudaStream_t s, const LatentParams& p, uint32_t T) {
   const LatentSpec& sp = p.spec;
+  constexpr uint32_t kM = kWarpsPerCta * 16;
   const uint32_t DQ = (sp.dim + sp.rot + 15u) & ~15u;
-  const size_t smem = mma_smem(DQ, DV);
-  cudaError_t e = cudaFuncSetAttribute(latent_prefill_mma_kernel<DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  const size_t smem = mma_smem(DQ, DV, kM, kTilePositions);
+  auto kern = latent_prefill_mma_kernel<DV, kWarpsPerCta, kTilePositions>;
+  cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return e;
   const int vec = sp.dim % 8 == 0 && sp.rot % 8 == 0 && sp.vdim % 8 == 0;
-  return launch_pdl(latent_prefill_mma_kernel<DV>, dim3((T + kM - 1) / kM * sp.heads), dim3(kThr), smem, s, prefill_pdl(), p, T, DQ, vec);
+  return launch_pdl(kern, dim3((T + kM - 1) / kM * sp.heads), dim3(kWarpsPerCta * 32), smem, s, prefill_pdl(), p, T, DQ, vec);
 }
 
 }  // namespace
 
 bool latent_prefill_mma_supported(const LatentSpec& s) {
   const uint32_t dv = value_width(s.vdim);
-  return dv && mma_smem((s.dim + s.rot + 15u) & ~15u, dv) <= 227 * 1024;
+  return dv && mma_smem((s.dim + s.rot + 15u) & ~15u, dv, kWarpsPerCta * 16, kTilePositions) <= 227 * 1024;
 }
 
 cudaError_t launch_latent_prefill_mma(cudaStream_t s, const LatentParams& p, uint32_t T) {

@@ -25,10 +25,21 @@ __device__ __forceinline__ float silu_f(float v) { return v / (1.0f + expf(-v));
 // One convolved channel at position pos, input rows from the ring
 __device__ __forceinline__ float conv_ring(const SsmParams& p, uint32_t pos, uint32_t ch) {
   const uint32_t K = p.spec.taps, ld = p.spec.in_rows();
+  const float* col = p.ring + p.spec.inner() + ch;
   float a = p.conv_b[ch];
-  for (uint32_t j = 0; j < K; ++j) {
-    const uint32_t back = K - 1 - j;
-    if (back <= pos) a = fmaf(p.conv_w[ch * K + j], __ldcg(p.ring + (size_t)((pos - back) % K) * ld + p.spec.inner() + ch), a);
+  uint32_t slot = (pos + 1) % K;  // row of the oldest tap's position
+  for (uint32_t j0 = 0; j0 < K; j0 += 4) {  // four taps' loads in flight together
+    float v[4], w[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const uint32_t j = j0 + i;
+      const bool in = j < K && K - 1 - j <= pos;
+      v[i] = in ? __ldcg(col + (size_t)slot * ld) : 0.f;
+      w[i] = in ? p.conv_w[ch * K + j] : 0.f;
+      slot = slot + 1 == K ? 0 : slot + 1;
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i) a = fmaf(w[i], v[i], a);
   }
   return silu_f(a);
 }
@@ -104,33 +115,59 @@ __global__ void __launch_bounds__(256) ssm_step_kernel(const SsmParams p) {
 }
 
 // ---- prompt path ------------------------------------------------------------------------------------------------------
-template <typename XT>
+// One channel per thread over kConvTB tokens. KT taps known at compile time: the inputs are requested together.
+constexpr uint32_t kConvTB = 16;
+template <typename XT, int KT>
 __global__ void __launch_bounds__(256) ssm_conv_kernel(const SsmParams p, uint32_t T) {
-  constexpr uint32_t TB = 8;  // tokens per thread
   const SsmSpec& sp = p.spec;
-  const uint32_t ch = blockIdx.x * 256 + threadIdx.x, CH = sp.channels(), ld = sp.in_rows(), K = sp.taps, inner = sp.inner();
+  const uint32_t ch = blockIdx.x * 256 + threadIdx.x, CH = sp.channels(), ld = sp.in_rows(), K = KT ? KT : sp.taps, inner = sp.inner();
   pdl_launch_dependents();
   pdl_wait();
   if (ch >= CH + sp.heads) return;
-  const uint32_t t0 = blockIdx.y * TB, t1 = min(T, t0 + TB);
+  const uint32_t t0 = blockIdx.y * kConvTB, t1 = min(T, t0 + kConvTB);
   if (ch >= CH) {
     const uint32_t h = ch - CH;
     for (uint32_t t = t0; t < t1; ++t) p.dt[(size_t)t * sp.heads + h] = softplus_f(p.in[(size_t)t * ld + inner + ch] + p.dt_bias[h]);
     return;
   }
-  XT* out = reinterpret_cast<XT*>(p.xbc);
+  XT* out = reinterpret_cast<XT*>(p.xbc) + ch;
+  const float* in = p.in + inner + ch;
   const float b = p.conv_b[ch];
-  for (uint32_t t = t0; t < t1; ++t) {
-    float a = b;
-    for (uint32_t j = 0; j < K; ++j) {
-      const uint32_t back = K - 1 - j;
-      float v = 0.f;
-      if (back <= t) v = p.in[(size_t)(t - back) * ld + inner + ch];
-      else if (back <= p.pos0 + t) v = p.ring[(size_t)((p.pos0 + t - back) % K) * ld + inner + ch];
-      a = fmaf(p.conv_w[ch * K + j], v, a);
+  auto past = [&](uint32_t t, uint32_t back) -> float {  // input `back` tokens before token t of the portion
+    if (back <= t) return in[(size_t)(t - back) * ld];
+    if (back <= p.pos0 + t) return p.ring[(size_t)((p.pos0 + t - back) % K) * ld + inner + ch];
+    return 0.f;
+  };
+  if constexpr (KT > 0) {
+    float v[kConvTB + KT - 1], w[KT];
+#pragma unroll
+    for (int j = 0; j < KT; ++j) w[j] = p.conv_w[ch * KT + j];
+#pragma unroll
+    for (int j = 0; j < KT - 1; ++j) v[j] = past(t0, KT - 1 - j);
+#pragma unroll
+    for (uint32_t i = 0; i < kConvTB; ++i) v[KT - 1 + i] = t0 + i < T ? in[(size_t)(t0 + i) * ld] : 0.f;
+#pragma unroll
+    for (uint32_t i = 0; i < kConvTB; ++i) {
+      float a = b;
+#pragma unroll
+      for (int j = 0; j < KT; ++j) a = fmaf(w[j], v[i + j], a);
+      if (t0 + i < T) store_as(out + (size_t)(t0 + i) * CH, silu_f(a));
     }
-    store_as(out + (size_t)t * CH + ch, silu_f(a));
+  } else {
+    for (uint32_t t = t0; t < t1; ++t) {
+      float a = b;
+      for (uint32_t j = 0; j < K; ++j) a = fmaf(p.conv_w[ch * K + j], past(t, K - 1 - j), a);
+      store_as(out + (size_t)t * CH, silu_f(a));
+    }
   }
+}
+
+template <typename XT>
+cudaError_t launch_conv(cudaStream_t s, const SsmParams& p, uint32_t T) {
+  const dim3 grid((p.spec.channels() + p.spec.heads + 255) / 256, (T + kConvTB - 1) / kConvTB);
+  auto kern = p.spec.taps == 2 ? ssm_conv_kernel<XT, 2> : p.spec.taps == 3 ? ssm_conv_kernel<XT, 3> : p.spec.taps == 4 ? ssm_conv_kernel<XT, 4>
+              : ssm_conv_kernel<XT, 0>;
+  return launch_pdl(kern, grid, dim3(256), 0, s, prefill_pdl(), p, T);
 }
 
 // the last rows of the portion into the ring, where decoding would have put them
@@ -224,26 +261,59 @@ __global__ void __launch_bounds__(256) ssm_scan_kernel(const SsmParams p, uint32
   }
 }
 
-template <typename OT>
+// A warp per (token, part). NQ > 0: parts of up to 128 NQ values in quads, kept in registers between the two passes.
+template <typename OT, int NQ>
 __global__ void __launch_bounds__(256) group_norm_rows_kernel(const float* __restrict__ y, const float* __restrict__ gain, float eps,
-                                                              uint32_t groups, uint32_t K, OT* __restrict__ out) {
-  __shared__ float red[8];
+                                                              uint32_t groups, uint32_t T, uint32_t K, OT* __restrict__ out) {
   pdl_launch_dependents();
   pdl_wait();
-  const uint32_t part = K / groups;
-  const float* yr = y + (size_t)blockIdx.x * K + (size_t)blockIdx.y * part;
-  const float* gr = gain + (size_t)blockIdx.y * part;
-  OT* o = out + (size_t)blockIdx.x * K + (size_t)blockIdx.y * part;
+  const uint32_t part = K / groups, lane = threadIdx.x & 31;
+  const size_t item = (size_t)blockIdx.x * 8 + (threadIdx.x >> 5);
+  if (item >= (size_t)T * groups) return;
+  const uint32_t g = (uint32_t)(item % groups);
+  const float* yr = y + item * part;
+  const float* gr = gain + (size_t)g * part;
+  OT* o = out + item * part;
   float ss = 0.f;
-  for (uint32_t i = threadIdx.x; i < part; i += 256) ss = fmaf(yr[i], yr[i], ss);
-  ss = warp_sum(ss);
-  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
-  __syncthreads();
-  float tot = 0.f;
+  if constexpr (NQ > 0) {
+    float4 v[NQ];
 #pragma unroll
-  for (int w = 0; w < 8; ++w) tot += red[w];
-  const float rms = sqrtf(__fdiv_rn(tot, (float)part) + eps);
-  for (uint32_t i = threadIdx.x; i < part; i += 256) store_as(o + i, __fmul_rn(__fdiv_rn(yr[i], rms), gr[i]));
+    for (int i = 0; i < NQ; ++i) {
+      const uint32_t at = (lane + 32 * i) * 4;
+      v[i] = at < part ? *reinterpret_cast<const float4*>(yr + at) : make_float4(0.f, 0.f, 0.f, 0.f);
+      ss = fmaf(v[i].x, v[i].x, ss);
+      ss = fmaf(v[i].y, v[i].y, ss);
+      ss = fmaf(v[i].z, v[i].z, ss);
+      ss = fmaf(v[i].w, v[i].w, ss);
+    }
+    const float rms = sqrtf(__fdiv_rn(warp_sum(ss), (float)part) + eps);
+#pragma unroll
+    for (int i = 0; i < NQ; ++i) {
+      const uint32_t at = (lane + 32 * i) * 4;
+      if (at < part) {
+        const float4 w = *reinterpret_cast<const float4*>(gr + at);
+        const float r[4] = {__fmul_rn(__fdiv_rn(v[i].x, rms), w.x), __fmul_rn(__fdiv_rn(v[i].y, rms), w.y),
+                            __fmul_rn(__fdiv_rn(v[i].z, rms), w.z), __fmul_rn(__fdiv_rn(v[i].w, rms), w.w)};
+        if constexpr (sizeof(OT) == 2) {
+          __nv_bfloat162 b[2] = {__floats2bfloat162_rn(r[0], r[1]), __floats2bfloat162_rn(r[2], r[3])};
+          *reinterpret_cast<uint2*>(o + at) = *reinterpret_cast<uint2*>(b);
+        } else {
+          *reinterpret_cast<float4*>(o + at) = make_float4(r[0], r[1], r[2], r[3]);
+        }
+      }
+    }
+  } else {
+    for (uint32_t i = lane; i < part; i += 32) ss = fmaf(yr[i], yr[i], ss);
+    const float rms = sqrtf(__fdiv_rn(warp_sum(ss), (float)part) + eps);
+    for (uint32_t i = lane; i < part; i += 32) store_as(o + i, __fmul_rn(__fdiv_rn(yr[i], rms), gr[i]));
+  }
+}
+
+template <typename OT>
+cudaError_t launch_norm(cudaStream_t s, const float* y, const float* gain, float eps, uint32_t groups, uint32_t T, uint32_t K, OT* out) {
+  const uint32_t part = K / groups;
+  auto kern = part % 4 || part > 1024 ? group_norm_rows_kernel<OT, 0> : part <= 512 ? group_norm_rows_kernel<OT, 4> : group_norm_rows_kernel<OT, 8>;
+  return launch_pdl(kern, dim3((unsigned)(((size_t)T * groups + 7) / 8)), dim3(256), 0, s, prefill_pdl(), y, gain, eps, groups, T, K, out);
 }
 
 template <typename XT>
@@ -272,9 +342,7 @@ cudaError_t launch_ssm_step(cudaStream_t s, const SsmParams& p, bool pdl) {
 
 cudaError_t launch_ssm_prefill(cudaStream_t s, const SsmParams& p, uint32_t T) {
   if (!T) return cudaErrorInvalidValue;
-  const dim3 cgrid((p.spec.channels() + p.spec.heads + 255) / 256, (T + 7) / 8);
-  cudaError_t e = p.xbc_dtype == 2 ? launch_pdl(ssm_conv_kernel<__nv_bfloat16>, cgrid, dim3(256), 0, s, prefill_pdl(), p, T)
-                                   : launch_pdl(ssm_conv_kernel<float>, cgrid, dim3(256), 0, s, prefill_pdl(), p, T);
+  cudaError_t e = p.xbc_dtype == 2 ? launch_conv<__nv_bfloat16>(s, p, T) : launch_conv<float>(s, p, T);
   if (e != cudaSuccess) return e;
   const uint32_t n = T < p.spec.taps ? T : p.spec.taps;
   e = launch_pdl(ssm_ring_kernel, dim3((p.spec.in_rows() + 255) / 256, n), dim3(256), 0, s, prefill_pdl(), p, T);
@@ -287,12 +355,9 @@ cudaError_t launch_ssm_prefill(cudaStream_t s, const SsmParams& p, uint32_t T) {
 
 cudaError_t launch_group_norm_rows(cudaStream_t s, const float* y, const float* gain, float eps, uint32_t groups, uint32_t T,
                                    uint32_t K, void* out, int out_dtype) {
-  if (!groups || K % groups || !T || groups > 65535) return cudaErrorInvalidValue;
-  const dim3 grid(T, groups);
-  if (out_dtype == 2)
-    return launch_pdl(group_norm_rows_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, prefill_pdl(), y, gain, eps, groups, K, (__nv_bfloat16*)out);
-  if (out_dtype == 0)
-    return launch_pdl(group_norm_rows_kernel<float>, grid, dim3(256), 0, s, prefill_pdl(), y, gain, eps, groups, K, (float*)out);
+  if (!groups || K % groups || !T) return cudaErrorInvalidValue;
+  if (out_dtype == 2) return launch_norm(s, y, gain, eps, groups, T, K, (__nv_bfloat16*)out);
+  if (out_dtype == 0) return launch_norm(s, y, gain, eps, groups, T, K, (float*)out);
   return cudaErrorInvalidValue;
 }
 

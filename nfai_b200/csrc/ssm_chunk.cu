@@ -102,6 +102,13 @@ __device__ __forceinline__ void chunk_sums(const SsmParams& p, uint32_t h, uint3
   }
 }
 
+// The chunk workspace: decays [chunks][heads], running sums (head, remainder, step size) [chunks][heads][3][kQ], then what
+// every chunk adds to the state [chunks][heads][vdim][state].
+__host__ __device__ inline size_t sums_offset(uint32_t heads, uint32_t nchunks) { return ((size_t)nchunks * heads + 3) & ~(size_t)3; }
+__host__ __device__ inline size_t added_offset(uint32_t heads, uint32_t nchunks) {
+  return sums_offset(heads, nchunks) + (size_t)nchunks * heads * 3 * kQ;
+}
+
 __host__ __device__ inline uint32_t pad16(uint32_t n) { return (n + 15u) & ~15u; }
 
 // ---- what a chunk adds to the state: [V][N] = sum_j (exp(c_last - c_j) dt_j x_j) B_j^T ----------------------------------------
@@ -122,6 +129,9 @@ __global__ void __launch_bounds__(kThr) ssm_chunk_state_kernel(const SsmParams p
   load_tile(Bs, LB, xbc + sp.inner() + (size_t)g * N, CH, t0, T, N, Np, vec);
   chunk_sums(p, h, t0, T, ch, cl, wt);
   __syncthreads();
+  float* const sums = p.chunk + sums_offset(sp.heads, gridDim.x) + ((size_t)chunk * sp.heads + h) * 3 * kQ;
+  for (uint32_t i = threadIdx.x; i < 3 * kQ; i += kThr) sums[i] = ch[i];  // for the output kernel (ch, cl and wt are contiguous)
+  __syncthreads();
   const float cend_h = ch[kQ - 1], cend_l = cl[kQ - 1];
   if (threadIdx.x < kQ) wt[threadIdx.x] *= expf((cend_h - ch[threadIdx.x]) + (cend_l - cl[threadIdx.x]));
   const size_t per_head = (size_t)V * N;
@@ -130,7 +140,7 @@ __global__ void __launch_bounds__(kThr) ssm_chunk_state_kernel(const SsmParams p
   if (threadIdx.x == 0) decays[(size_t)chunk * sp.heads + h] = expf(cend_h + cend_l);
   wait_copies();
   __syncthreads();
-  float* const out = p.chunk + (((size_t)nchunks * sp.heads + 3) & ~(size_t)3) + ((size_t)chunk * sp.heads + h) * per_head;
+  float* const out = p.chunk + added_offset(sp.heads, nchunks) + ((size_t)chunk * sp.heads + h) * per_head;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, lm = lane >> 3, lr = lane & 7, qr = lane >> 2, qc = (lane & 3) * 2;
   const uint32_t ntiles = (Np + 63) / 64, tiles = Vp / 16 * ntiles;
   for (uint32_t tile = warp; tile < tiles; tile += kThr / 32) {
@@ -174,29 +184,45 @@ __global__ void __launch_bounds__(kThr) ssm_chunk_state_kernel(const SsmParams p
 }
 
 // ---- states before every chunk, in place of what the chunks add; the state after the last one into p.S -------------------------
-__global__ void __launch_bounds__(256) ssm_chunk_pass_kernel(const SsmParams p, const uint32_t nchunks) {
+__global__ void __launch_bounds__(128) ssm_chunk_pass_kernel(const SsmParams p, const uint32_t nchunks) {
   pdl_launch_dependents();
   pdl_wait();
   const size_t per_head = (size_t)p.spec.vdim * p.spec.state, total = per_head * p.spec.heads;
-  const size_t i = (size_t)blockIdx.x * 256 + threadIdx.x;
-  if (i >= total) return;
-  const uint32_t h = (uint32_t)(i / per_head);
   const float* decays = p.chunk;
-  float* add = p.chunk + (((size_t)nchunks * p.spec.heads + 3) & ~(size_t)3);
-  float s = p.pos0 > 0 ? p.S[i] : 0.f;
-  for (uint32_t c0 = 0; c0 < nchunks; c0 += 8) {
-    float a[8];
+  float* add = p.chunk + added_offset(p.spec.heads, nchunks);
+  auto walk = [&](auto* s_ptr, auto* a_ptr, size_t stride, uint32_t h, auto&& step) {
+    auto s = *s_ptr;
+    if (p.pos0 == 0) step(s, 0.f, s, true);
+    for (uint32_t c0 = 0; c0 < nchunks; c0 += 8) {
+      decltype(s) a[8];
+      float d[8];
 #pragma unroll
-    for (int j = 0; j < 8; ++j)
-      if (c0 + j < nchunks) a[j] = add[(size_t)(c0 + j) * total + i];
+      for (int j = 0; j < 8; ++j)
+        if (c0 + j < nchunks) {
+          a[j] = a_ptr[(size_t)(c0 + j) * stride];
+          d[j] = decays[(size_t)(c0 + j) * p.spec.heads + h];
+        }
 #pragma unroll
-    for (int j = 0; j < 8; ++j)
-      if (c0 + j < nchunks) {
-        add[(size_t)(c0 + j) * total + i] = s;
-        s = fmaf(decays[(size_t)(c0 + j) * p.spec.heads + h], s, a[j]);
-      }
+      for (int j = 0; j < 8; ++j)
+        if (c0 + j < nchunks) {
+          a_ptr[(size_t)(c0 + j) * stride] = s;
+          step(s, d[j], a[j], false);
+        }
+    }
+    *s_ptr = s;
+  };
+  const size_t i = (size_t)blockIdx.x * 128 + threadIdx.x;
+  if (per_head % 4 == 0) {
+    if (i * 4 >= total) return;
+    walk(reinterpret_cast<float4*>(p.S) + i, reinterpret_cast<float4*>(add) + i, total / 4, (uint32_t)(i * 4 / per_head),
+         [](float4& s, float d, const float4& a, bool zero) {
+           if (zero) s = make_float4(0.f, 0.f, 0.f, 0.f);
+           else s = make_float4(fmaf(d, s.x, a.x), fmaf(d, s.y, a.y), fmaf(d, s.z, a.z), fmaf(d, s.w, a.w));
+         });
+  } else {
+    if (i >= total) return;
+    walk(p.S + i, add + i, total, (uint32_t)(i / per_head), [](float& s, float d, const float& a, bool zero) { s = zero ? 0.f : fmaf(d, s, a); });
   }
-  p.S[i] = s;
 }
 
 // ---- outputs ---------------------------------------------------------------------------------------------------------------------
@@ -218,11 +244,18 @@ __global__ void __launch_bounds__(kThr, VT <= 64 ? 2 : 1) ssm_chunk_out_kernel(c
   pdl_launch_dependents();
   pdl_wait();
   const __nv_bfloat16* xbc = reinterpret_cast<const __nv_bfloat16*>(p.xbc);
+  // the gate's rows are needed last: have them on their way from memory
+  for (uint32_t i = threadIdx.x; i < kQ * ((V * 4 + 127) / 128); i += kThr) {
+    const uint32_t lines = (V * 4 + 127) / 128, r = i / lines, l = i - r * lines;
+    if (t0 + r < T) asm volatile("prefetch.global.L2 [%0];" ::"l"(p.in + (size_t)(t0 + r) * sp.in_rows() + (size_t)h * V + l * 32));
+  }
   load_tile(Cs, LB, xbc + inner + (size_t)(sp.groups + g) * N, CH, t0, T, N, Np, vec);
   load_tile(Xs, LX, xbc + (size_t)h * V, CH, t0, T, V, VT, vec);
-  chunk_sums(p, h, t0, T, ch, cl, dts);
+  const float* sums = p.chunk + sums_offset(sp.heads, gridDim.x) + ((size_t)chunk * sp.heads + h) * 3 * kQ;
+  for (uint32_t i = threadIdx.x; i < 3 * kQ; i += kThr) ch[i] = sums[i];  // ch, cl and dts are contiguous
   const size_t per_head = (size_t)V * N;
-  const float* S0 = p.chunk + (((size_t)gridDim.x * sp.heads + 3) & ~(size_t)3) + ((size_t)chunk * sp.heads + h) * per_head;
+  const float* S0 = p.chunk + added_offset(sp.heads, gridDim.x) + ((size_t)chunk * sp.heads + h) * per_head;
+#pragma unroll 4
   for (uint32_t i = threadIdx.x; i < VT * (Np / 2); i += kThr) {
     const uint32_t v = i / (Np / 2), n = (i - v * (Np / 2)) * 2;
     const float a = v < V && n < N ? S0[(size_t)v * N + n] : 0.f, b = v < V && n + 1 < N ? S0[(size_t)v * N + n + 1] : 0.f;
@@ -355,7 +388,7 @@ bool ssm_chunk_supported(const SsmSpec& s) {
 size_t ssm_chunk_floats(const SsmSpec& s, uint32_t T) {
   if (!ssm_chunk_supported(s)) return 0;
   const size_t n = (T + kQ - 1) / kQ;
-  return ((n * s.heads + 3) & ~(size_t)3) + n * s.heads * s.vdim * s.state;
+  return added_offset(s.heads, (uint32_t)n) + n * s.heads * s.vdim * s.state;
 }
 
 cudaError_t launch_ssm_chunked(cudaStream_t s, const SsmParams& p, uint32_t T) {
@@ -370,7 +403,7 @@ cudaError_t launch_ssm_chunked(cudaStream_t s, const SsmParams& p, uint32_t T) {
   e = launch_pdl(ssm_chunk_state_kernel, dim3(nchunks, sp.heads), dim3(kThr), smem, s, prefill_pdl(), p, T, vec);
   if (e != cudaSuccess) return e;
   const size_t total = (size_t)sp.heads * sp.vdim * sp.state;
-  e = launch_pdl(ssm_chunk_pass_kernel, dim3((unsigned)((total + 255) / 256)), dim3(256), 0, s, prefill_pdl(), p, nchunks);
+  e = launch_pdl(ssm_chunk_pass_kernel, dim3((unsigned)(((sp.vdim * sp.state % 4 ? total : total / 4) + 127) / 128)), dim3(128), 0, s, prefill_pdl(), p, nchunks);
   if (e != cudaSuccess) return e;
   switch (out_width(sp.vdim)) {
     case 32: return launch_out<32>(s, p, T, nchunks, vec);
