@@ -1477,7 +1477,7 @@ int nfai_model_set_prefetch(nfai_model* m, uint64_t lookahead_bytes, uint64_t ex
 
 int nfai_step_launches(const nfai_model* m, int* out) {
   if (!m || !out) return fail(m ? m->ctx : nullptr, NFAI_ERR_ARG, "null argument");
-  *out = m->launches_full;
+  *out = m->plan && !m->ctx->use_graph ? plan_step_launches(m) : m->launches_full;
   return NFAI_OK;
 }
 

@@ -1,7 +1,7 @@
 // Latent attention: per position one RMS-normed latent c (rank values) and one rotated key part shared by all heads are
 // cached; a head's keys and values are linear maps of c. Sliding window, per-element sigmoid gate on the output.
 //
-// Decode (latent_decode_kernel) never expands a key or a value. A head's query is pulled back through its key map
+// Decode (latent_decode_kernel here for true float32 and any sizes; latent_decode_mma.cu for bfloat16 caches) never expands a key or a value. A head's query is pulled back through its key map
 // (q_lat = W_uk^T q), scores are q_lat . c + q_rot . k_rot, the weighted sum is taken over the latents themselves and only
 // the finished sum goes through the value map. One thread-block cluster works on one head; its CTAs
 //   1. each make a slice of q_lat and write it into every CTA of the cluster (distributed shared memory),
@@ -15,70 +15,13 @@
 // (float32, and head sizes the former does not take) run causal windowed attention over them.
 #include <string>
 
-#include "attn_core.cuh"
-#include "plan_kernels.h"
+#include "latent_common.cuh"
 
 namespace nfai {
 
 namespace {
 
-constexpr float kNeg = attn_detail::kNegBig;
-
-__device__ __forceinline__ float sigmoid_f(float v) { return 1.0f / (1.0f + expf(-v)); }
-
-// Rotated entry i of a key/query part held in `src`: entry i < half pairs with i + half; entries past 2 half pass.
-__device__ __forceinline__ float rotated(const float* src, uint32_t i, uint32_t dims, const float2* cs) {
-  const uint32_t half = dims >> 1;
-  if (i >= dims) return src[i];
-  const uint32_t j = i < half ? i : i - half;
-  const float2 r = cs[j];
-  const float u = src[j], v = src[j + half];
-  return i < half ? __fsub_rn(__fmul_rn(u, r.x), __fmul_rn(v, r.y)) : __fadd_rn(__fmul_rn(v, r.x), __fmul_rn(u, r.y));
-}
-
-template <typename T>
-__device__ __forceinline__ T cast_to(float v) {
-  T t;
-  store_as(&t, v);
-  return t;
-}
-
-// V consecutive elements -> float
-template <typename T, int V>
-__device__ __forceinline__ void load_vec(const T* p, float (&f)[V]) {
-  if constexpr (V > 1) {
-    static_assert(V == WeightVec<T>::kElems, "16-byte vectors");
-    WeightVec<T>::unpack(*reinterpret_cast<const uint4*>(p), f);
-  } else {
-    f[0] = to_float(*p);
-  }
-}
-
-__device__ __forceinline__ uint32_t cluster_rank() {
-  uint32_t r;
-  asm volatile("mov.u32 %0, %%cluster_ctarank;" : "=r"(r));
-  return r;
-}
-__device__ __forceinline__ void cluster_arrive() { asm volatile("barrier.cluster.arrive.release;" ::: "memory"); }
-__device__ __forceinline__ void cluster_wait() { asm volatile("barrier.cluster.wait.acquire;" ::: "memory"); }
-// address of the same shared-memory location in CTA `rank` of the cluster
-__device__ __forceinline__ uint32_t peer_addr(const void* p, uint32_t rank) {
-  uint32_t a = (uint32_t)__cvta_generic_to_shared(p), r;
-  asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(r) : "r"(a), "r"(rank));
-  return r;
-}
-__device__ __forceinline__ void st_peer(uint32_t addr, float v) { asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(addr), "f"(v) : "memory"); }
-__device__ __forceinline__ float ld_peer(uint32_t addr) {
-  float v;
-  asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(addr) : "memory");
-  return v;
-}
-__device__ __forceinline__ void cp16(uint32_t dst, const void* src, uint32_t bytes) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(bytes) : "memory");
-}
-__device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N>
-__device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+using namespace latent_detail;
 
 // ---- decode -------------------------------------------------------------------------------------------------------------
 constexpr int kDT = 256;   // threads per CTA
@@ -550,9 +493,25 @@ bool latent_supported(const LatentSpec& s, int dtype, std::string* why) {
   return true;
 }
 
-cudaError_t launch_latent_decode(cudaStream_t s, const LatentParams& p, bool pdl) {
-  // CTAs per head: as many as keep the grid within one wave, but no more than there are blocks of rows to share
+// latent_decode_mma.cu
+bool latent_decode_mma_supported(const LatentSpec& s);
+size_t latent_decode_mma_scratch(const LatentSpec& s, uint32_t ctx, size_t* tiles_bytes);
+cudaError_t launch_latent_decode_mma(cudaStream_t s, const LatentParams& p, uint32_t rows, bool pdl, int* launches);
+
+static bool decode_on_tensor_cores(const LatentSpec& s, int dtype) {
+  static const bool on = env_int("NFAI_LATENT_MMA", 1) != 0;
+  return dtype == 2 && on && latent_decode_mma_supported(s);
+}
+
+size_t latent_decode_scratch(const LatentSpec& s, int dtype, uint32_t ctx) {
+  return decode_on_tensor_cores(s, dtype) ? latent_decode_mma_scratch(s, ctx, nullptr) : 0;
+}
+
+cudaError_t launch_latent_decode(cudaStream_t s, const LatentParams& p, bool pdl, int* launches) {
   const uint32_t rows = p.spec.window && p.spec.window < p.ctx ? p.spec.window : p.ctx;
+  if (decode_on_tensor_cores(p.spec, p.dtype)) return launch_latent_decode_mma(s, p, rows, pdl, launches);
+  if (launches) ++*launches;
+  // CTAs per head: as many as keep the grid within one wave, but no more than there are blocks of rows to share
   uint32_t C = 8;
   while (C > 1 && (C * p.spec.heads > sm_count() || (rows + C - 1) / C < 16)) C >>= 1;
   if (p.dtype == 0) return vec_of(p.spec, 0) > 1 ? launch_decode_t<float, 4>(s, p, C, pdl) : launch_decode_t<float, 1>(s, p, C, pdl);

@@ -53,6 +53,7 @@ struct LatentParams {
   uint32_t pos0 = 0;                // prompt path (and decode without state): position of the first token
   // decode
   float* out = nullptr;             // [heads*vdim], gated
+  void* scratch = nullptr;          // latent_decode_scratch bytes, zero-filled once
   // prompt path
   void* q = nullptr;                // [T][heads*(dim+rot)] of dtype, rotated
   const void* kv = nullptr;         // [rows][heads*dim | heads*vdim] of dtype; row 0 is position kv_pos0
@@ -60,7 +61,9 @@ struct LatentParams {
   void* ao = nullptr;               // [T][heads*vdim] of dtype, gated
 };
 bool latent_supported(const LatentSpec& s, int dtype, std::string* why);
-cudaError_t launch_latent_decode(cudaStream_t s, const LatentParams& p, bool pdl);
+size_t latent_decode_scratch(const LatentSpec& s, int dtype, uint32_t ctx);
+// Adds the number of kernels it launched to *launches (may be null).
+cudaError_t launch_latent_decode(cudaStream_t s, const LatentParams& p, bool pdl, int* launches);
 // Norm and rotate what the projection of T tokens left: cache rows pos0 .. pos0+T-1 and p.q.
 cudaError_t launch_latent_prep(cudaStream_t s, const LatentParams& p, uint32_t T);
 // Windowed causal attention of the T tokens over the expanded keys and values, gated.

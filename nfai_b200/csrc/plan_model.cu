@@ -4,7 +4,7 @@
 //
 // Decode step, per layer (H = width, S = streams):
 //   latent attention   GEMV [q | latent, key part | gate] (norm in its prologue)
-//                      latent_decode_kernel (query to latents, window, values, gate; cache row)
+//                      latent_decode (query to latents, window, values, gate; cache row)
 //                      GEMV o, whose epilogue writes all S streams and forms the next sublayer's input
 //   state space        GEMV in-projection into the ring row of this position
 //                      ssm_step_kernel (convolution, step size, state, skip, gate)
@@ -47,6 +47,7 @@ struct LayerState {
   // latent attention
   char* c = nullptr;
   char* kr = nullptr;
+  void* scratch = nullptr;
   float2* rope = nullptr;
   // state space
   float* ring = nullptr;
@@ -77,6 +78,7 @@ struct PlanModel {
   float* mix = nullptr;  // [max in_rows]
   float* ao = nullptr;   // [max out_cols]
   float* hbuf = nullptr; // [max ff]
+  int step_launches = 0;
   // prompt passes
   bool batched = false;
   uint32_t chunk = 0;
@@ -337,7 +339,7 @@ int plan_finalize(nfai_model* m) {
   Arena a;
   const CommonOffsets common = place_common(m, a);
   // per layer: caches and states; one (cos, sin) table per distinct rotation
-  struct Off { size_t c = 0, kr = 0, rope = 0, ring = 0, S = 0; };
+  struct Off { size_t c = 0, kr = 0, scratch = 0, rope = 0, ring = 0, S = 0; };
   std::vector<Off> off(hp.L);
   std::map<std::pair<uint32_t, float>, size_t> ropes;
   for (uint32_t i = 0; i < hp.L; ++i) {
@@ -345,6 +347,7 @@ int plan_finalize(nfai_model* m) {
     if (l.mixer == MIXER_LATENT) {
       off[i].c = a.take((size_t)hp.ctx * l.latent.rank * as);
       off[i].kr = a.take((size_t)hp.ctx * l.latent.rot * as);
+      off[i].scratch = a.take(latent_decode_scratch(l.latent, P->act_dtype, hp.ctx));
       const std::pair<uint32_t, float> key(l.latent.rope_dims, l.latent.rope_base);
       auto r = ropes.find(key);
       if (r == ropes.end()) r = ropes.emplace(key, a.take((size_t)hp.ctx * (key.first / 2) * sizeof(float2) + 16)).first;
@@ -400,6 +403,7 @@ int plan_finalize(nfai_model* m) {
     if (pl.layers[i].mixer == MIXER_LATENT) {
       s.c = base + off[i].c;
       s.kr = base + off[i].kr;
+      s.scratch = base + off[i].scratch;
       s.rope = (float2*)(base + off[i].rope);
     } else {
       s.ring = (float*)(base + off[i].ring);
@@ -552,6 +556,7 @@ LatentParams latent_params(nfai_model* m, uint32_t l) {
   p.kr_cache = P->st[l].kr;
   p.dtype = P->act_dtype;
   p.ctx = m->hp.ctx;
+  p.scratch = P->st[l].scratch;
   return p;
 }
 
@@ -570,18 +575,19 @@ SsmParams ssm_params(nfai_model* m, uint32_t l) {
   return p;
 }
 
-cudaError_t launch_mixer_step(nfai_model* m, uint32_t l, bool pdl) {
+cudaError_t launch_mixer_step(nfai_model* m, uint32_t l, bool pdl, int* launches) {
   PlanModel* P = m->plan.get();
   if (P->plan.layers[l].mixer == MIXER_LATENT) {
     LatentParams p = latent_params(m, l);
     p.in = P->mix;
     p.state = m->state;
     p.out = P->ao;
-    return launch_latent_decode(m->ctx->stream, p, pdl);
+    return launch_latent_decode(m->ctx->stream, p, pdl, launches);
   }
   SsmParams p = ssm_params(m, l);
   p.state = m->state;
   p.y = P->ao;
+  if (launches) ++*launches;
   return launch_ssm_step(m->ctx->stream, p, pdl);
 }
 
@@ -622,7 +628,7 @@ cudaError_t plan_record_step(nfai_model* m, bool with_head, bool from_prompt, in
   uint32_t sub = 0;
   for (uint32_t l = 0; l < hp.L; ++l) {
     STEP(launch_gemv(s, wdt, 0, EPI_STORE, in_params(m, l), m->tune_qkv, pdl));
-    STEP(launch_mixer_step(m, l, pdl));
+    if ((e = launch_mixer_step(m, l, pdl, &n)) != cudaSuccess) return e;
     STEP(launch_gemv(s, wdt, 0, EPI_HYPER, out_params(m, l, sub++), m->tune_o, pdl));
     if (P->plan.layers[l].has_mlp) {
       STEP(launch_gemv(s, wdt, 0, EPI_GATED, gateup_params(m, l), m->tune_gateup, pdl));
@@ -638,14 +644,12 @@ cudaError_t plan_record_step(nfai_model* m, bool with_head, bool from_prompt, in
   }
 #undef STEP
   if (launches) *launches = n;
+  if (with_head) P->step_launches = n;
   return cudaSuccess;
 }
 
-int plan_step_launches(const nfai_model* m) {
-  int n = 3;
-  for (const PlanLayer& l : m->plan->plan.layers) n += l.has_mlp ? 5 : 3;
-  return n;
-}
+// (without graphs: known after the first recorded step)
+int plan_step_launches(const nfai_model* m) { return m->plan->step_launches; }
 
 // ---- prompt passes ----------------------------------------------------------------------------------------------------------------
 bool plan_batched(const nfai_model* m) { return m->plan->batched && m->plan->chunk >= 2; }
@@ -935,7 +939,7 @@ cudaError_t plan_profile_launch(nfai_model* m, int which, int iter) {
     case 1: return launch_gemv(s, wdt, 0, EPI_HYPER, down_params(m, l, sub + 1), m->tune_down, false);
     case 2: case 6: return launch_gemv(s, wdt, 0, EPI_STORE, in_params(m, l), m->tune_qkv, false);
     case 3: case 8: return launch_gemv(s, wdt, 0, EPI_HYPER, out_params(m, l, sub), m->tune_o, false);
-    default: return launch_mixer_step(m, l, false);
+    default: return launch_mixer_step(m, l, false, nullptr);
   }
 }
 
