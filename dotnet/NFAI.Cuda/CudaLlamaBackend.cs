@@ -17,6 +17,16 @@ public sealed unsafe class CudaLlamaBackend : IDisposable
         Native.Check(Native.nfai_model_create(ctx.Handle, in hp, out model), ctx.Handle);
     }
 
+    // A model folder (config.json + model.safetensors) of one of the layer-plan architectures; every method below works on
+    // it as on a Llama model, except that a position can only be rewound to 0 or through a snapshot.
+    public CudaLlamaBackend(CudaContext ctx, string modelFolder, uint kvCacheSize, NfaiDType weights = NfaiDType.BF16)
+    {
+        this.ctx = ctx;
+        Native.Check(Native.nfai_model_load_dir(ctx.Handle, modelFolder, kvCacheSize, (int)weights, out model), ctx.Handle);
+        Native.Check(Native.nfai_model_get_hparams(model, out NfaiHParams hp), ctx.Handle);
+        Vocab = hp.V;
+    }
+
     // Streams one tensor exactly as the reference does for a shader property: the chunks GetDataRaw yields
     // (halves already widened to float32, NFAI.Core/AbstractComputeCollection.cs:36-79) go to the device.
     public void Upload(AbstractComputeCollection tensor, IEnumerable<byte[]> rawChunks, bool chunksAreFloat32)

@@ -5,7 +5,7 @@ using System.Runtime.InteropServices;
 namespace NFAI.Cuda;
 
 public enum NfaiStatus { Ok = 0, Arg = 1, State = 2, Oom = 3, Cuda = 4, Nccl = 5, ContextFull = 6, Timeout = 7 }
-public enum NfaiDType { F32 = 0, F16 = 1 }
+public enum NfaiDType { F32 = 0, F16 = 1, BF16 = 2 }
 
 [StructLayout(LayoutKind.Sequential)]
 public struct NfaiHParams
@@ -35,6 +35,12 @@ internal static unsafe partial class Native
     [DllImport(Lib)] internal static extern int nfai_model_finalize(IntPtr model);
     [DllImport(Lib, CharSet = CharSet.Ansi)] internal static extern int nfai_model_load_gguf(IntPtr ctx, string path, uint kvCacheSize, int kvDType, out IntPtr model);
     [DllImport(Lib, CharSet = CharSet.Ansi)] internal static extern int nfai_gguf_probe(string path, uint kvCacheSize, out NfaiHParams hp, byte* errOut, nuint errBytes);
+    // models described by a configuration (layer plans)
+    [DllImport(Lib)] internal static extern int nfai_config_probe(byte[] configJson, nuint len, out NfaiHParams hp, byte* tensorsOut, nuint cap, out nuint n, byte* errOut, nuint errBytes);
+    [DllImport(Lib)] internal static extern int nfai_model_create_from_config(IntPtr ctx, byte[] configJson, nuint len, uint kvCacheSize, int weightDType, out IntPtr model);
+    [DllImport(Lib, CharSet = CharSet.Ansi)] internal static extern int nfai_model_load_dir(IntPtr ctx, string dir, uint kvCacheSize, int weightDType, out IntPtr model);
+    [DllImport(Lib)] internal static extern int nfai_forward(IntPtr model, uint* tokens, int n, uint* want, int nWant, float* logits);
+    [DllImport(Lib)] internal static extern int nfai_op_gemm(IntPtr ctx, void* a, void* w, int dtype, uint m, uint n, uint k, float* c);
     [DllImport(Lib)] internal static extern int nfai_model_get_hparams(IntPtr model, out NfaiHParams hp);
     [DllImport(Lib)] internal static extern int nfai_op_gemm_f16(IntPtr ctx, void* a, void* w, uint m, uint n, uint k, float* c);
     [DllImport(Lib)] internal static extern int nfai_model_destroy(IntPtr model);

@@ -265,6 +265,31 @@ def test_window_edges(cuda_ctx, window, dtype):
     m.Dispose()
 
 
+@pytest.mark.parametrize("heads,dim,rot,vdim,rank,window", [(20, 16, 16, 24, 64, 50), (17, 8, 32, 8, 48, 300), (33, 8, 16, 16, 32, 7)])
+@pytest.mark.parametrize("dtype", ["f32", "bf16"])
+def test_many_heads(cuda_ctx, heads, dim, rot, vdim, rank, window, dtype):
+    """More heads than one operand tile of the decode kernels holds."""
+    cfg = U.config([U.layer(U.latent(heads, dim, rot, vdim, rank, window))], 40, 64, 2)
+    alone(cuda_ctx, cfg, U.weights(cfg, heads), np.random.default_rng(1).integers(0, 64, 110).tolist(), dtype)
+
+
+def test_runs_of_several_stages(cuda_ctx):
+    """A window so long, for so many heads, that a CTA of the decode kernel walks its share of the cache in several stages."""
+    cfg = U.config([U.layer(U.latent(100, 4, 16, 4, 272, 760))], 40, 64, 2)
+    W = U.weights(cfg, 9)
+    W64 = {k: v.astype(np.float64) for k, v in W.items()}
+    toks = np.random.default_rng(2).integers(0, 64, 790).tolist()
+    narrow = json.loads(json.dumps(cfg))
+    narrow["layers"][0]["mixer"]["mask"]["size"] = 1  # what one layer leaves in the cache does not depend on its window
+    st = P.State(narrow)
+    P.forward(narrow, W64, toks[:740], st, cache=bf16)
+    ref = P.forward(cfg, W64, toks[740:], st, cache=bf16)
+    m = build(cuda_ctx, cfg, W, "bf16", 800)
+    m.forward(toks[:740])
+    assert U.error([m.decode(t)[0] for t in toks[740:]], ref) < 1e-3
+    m.Dispose()
+
+
 def test_cached_rows(cuda_ctx):
     """The cache holds the normed latent and the rotated key part, whichever path wrote it."""
     cfg, W, toks, _, _ = plain("even")
