@@ -158,11 +158,14 @@ int nfai_model_get_hparams(const nfai_model* m, nfai_hparams* out);
 /* ---- models described by a configuration (layer plans) -------------------------------------------------------
  * A model folder holds config.json, whose "architecture" names the design and whose "layers" list every layer's mixer
  * (its kind and sizes) and feed-forward, and model.safetensors. Known architectures: "Tometar" (hyper-connected
- * residual streams, latent attention with a sliding window, Mamba-2 layers, relu-gated feed-forwards). The handle is an
+ * residual streams, latent attention with a sliding window, Mamba-2 layers, relu-gated feed-forwards) and "Tutizen"
+ * (post-norm residual, grouped-query attention with head norms, distance bias, head gates and borrowed keys and values,
+ * clamped gated feed-forwards, dense or routed over experts). The handle is an
  * nfai_model like any other: prefill, decode, greedy and sampled loops, snapshots and taps work on it. Differences:
  * nfai_set_position only goes to 0 or the current position (recurrent state), one GPU, the cache has the weights' type,
  * nfai_read_kv returns the latent (kv_rank floats) as k and the shared rotated key part (rot_dim floats) as v of a latent
- * attention layer, nfai_read_hidden the sum of the streams. weight_dtype: NFAI_BF16 (served precision) or NFAI_F32 (true
+ * attention layer, and the normed heads (kv_heads * dim and kv_heads * vdim floats) of a grouped-query layer or the layer it
+ * borrows from; nfai_read_hidden the sum of the streams. weight_dtype: NFAI_BF16 (served precision) or NFAI_F32 (true
  * 32-bit everywhere). No counterpart in the reference, whose one model family is Llama
  * (NFAI.Models.Llama3/LlamaModelFactory.cs:36-44). */
 int nfai_model_create_from_config(nfai_ctx* ctx, const char* config_json, size_t len, uint32_t kv_cache_size,
@@ -254,8 +257,9 @@ int nfai_read_hidden(nfai_model* m, uint32_t layer, float* out);
  * events; launch i uses layer (i mod L)'s weights so that consecutive launches read different HBM.
  * which: 0 = FFN gate/up GEMV (+RMSNorm, +SiLU*up), 1 = FFN down GEMV (+residual), 2 = QKV GEMV (+RMSNorm,+RoPE),
  *        3 = O-projection GEMV (+residual), 4 = LM-head GEMV (+RMSNorm, +arg-max partials), 5 = attention.
- *        Layer-plan models: 0 and 1 feed-forward, 2 input projection, 3 output projection and 5 attention of latent
- *        attention layers, 4 LM head, 6 input projection, 7 step and 8 output projection of state space layers.
+ *        Layer-plan models: 0 and 1 dense feed-forward, 2 input projection, 3 output projection and 5 attention of
+ *        attention layers, 4 LM head, 6 input projection, 7 step and 8 output projection of state space layers, 9 shared
+ *        gate/up with the router, 10 gate/up of the chosen experts and 11 down of routed feed-forwards.
  * avg_ms receives the mean duration of one launch; bytes_per_launch the algorithmic bytes it must move. */
 int nfai_profile_kernel(nfai_model* m, int which, int iters, float* avg_ms, uint64_t* bytes_per_launch);
 

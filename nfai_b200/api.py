@@ -365,8 +365,32 @@ class PlannedModel(CausalModel):
         self.weight_dtype = self.kv_dtype = _dtype_name(self.hp.weight_dtype)
         self.ModelName = name
 
-    KERNELS = {"ffn_gate_up": 0, "ffn_down": 1, "latent_in": 2, "latent_out": 3, "lm_head": 4, "latent_attention": 5,
-               "ssm_in": 6, "ssm_step": 7, "ssm_out": 8}
+    @property
+    def KERNELS(self) -> Dict[str, int]:  # noqa: N802
+        """Selectors of the decode-step kernels this model's layers have."""
+        layers = self.config["layers"]
+        kinds = {(layer.get("mlp") or {}).get("kind") for layer in layers}
+        out = {"lm_head": 4}
+        if "dense" in kinds:
+            out.update(ffn_gate_up=0, ffn_down=1)
+        if "moe" in kinds:
+            out.update(shared_gate_up_router=9, expert_gate_up=10, expert_down=11)
+        for layer in layers:
+            if layer["type"] == "mamba2":
+                out.update(ssm_in=6, ssm_step=7, ssm_out=8)
+            elif layer["type"] == "latent_attention":
+                out.update(latent_in=2, latent_out=3, latent_attention=5)
+            else:
+                out.update(attn_in=2, attn_out=3, attention=5)
+        return out
+
+    def read_kv(self, layer: int, pos: int) -> Tuple[np.ndarray, np.ndarray]:
+        """Cached keys [kv_heads][dim] and values [kv_heads][vdim] of one position of an attention layer (of the layer it
+        borrows them from, if it does)."""
+        m = self.config["layers"][layer]["mixer"]
+        k, v = np.empty((m["kv_heads"], m["dim"]), np.float32), np.empty((m["kv_heads"], m["vdim"]), np.float32)
+        check(self._lib.nfai_read_kv(self.handle, layer, pos, self._fp(k), self._fp(v)), self.ctx.handle)
+        return k, v
 
     def read_latent(self, layer: int, pos: int) -> Tuple[np.ndarray, np.ndarray]:
         """Cached latent and rotated key part of one position of a latent attention layer."""

@@ -1486,7 +1486,7 @@ int nfai_profile_kernel(nfai_model* m, int which, int iters, float* avg_ms, uint
   if (rc) return rc;
   nfai_ctx* c = m->ctx;
   const nfai_hparams& hp = m->hp;
-  if (iters <= 0 || which < 0 || which > (m->plan ? 8 : 5)) return fail(c, NFAI_ERR_ARG, "bad kernel selector or iteration count");
+  if (iters <= 0 || which < 0 || which > (m->plan ? 11 : 5)) return fail(c, NFAI_ERR_ARG, "bad kernel selector or iteration count");
   if (which == 5 && m->pos == 0) return fail(c, NFAI_ERR_STATE, "attention profiling needs at least one cached position");
   const int wdt = hp.weight_dtype, kvdt = hp.kv_dtype;
   const size_t ws = dtype_size(wdt), kvs = dtype_size(kvdt);

@@ -66,7 +66,12 @@ __device__ __forceinline__ void epilogue_pair(const GemmEpilogue& ep, uint32_t m
       break;
     }
     case GEMM_EPI_GATED: {  // columns (2j, 2j+1) = (gate_j, up_j); h_j = up * act(gate)
-      if (n + 1 < N) store_operand(ep, (size_t)m * (N / 2) + (n >> 1), gated(ep.act, a + aux.x, b + aux.y));
+      if (ep.gated_cols && n >= ep.gated_cols) {  // plain columns behind the gated ones (both counts are even)
+        *reinterpret_cast<float2*>(ep.out_f32 + (size_t)m * (N - ep.gated_cols) + (n - ep.gated_cols)) = make_float2(a, b);
+        break;
+      }
+      if (n + 1 < N)
+        store_operand(ep, (size_t)m * ((ep.gated_cols ? ep.gated_cols : N) / 2) + (n >> 1), gated(ep.act, a + aux.x, b + aux.y, ep.act_limit));
       break;
     }
     case GEMM_EPI_STORE_ACT: {  // plain store in the operand type of the next product

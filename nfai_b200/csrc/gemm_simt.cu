@@ -10,13 +10,23 @@ namespace {
 
 constexpr int kT = 64, kKS = 16;
 
-template <typename T>
+template <typename T, bool GROUPED>
 __global__ void __launch_bounds__(256) gemm_simt_kernel(const T* __restrict__ A, const T* __restrict__ W, uint32_t M, uint32_t N,
-                                                        uint32_t K, const GemmEpilogue ep) {
+                                                        uint32_t K, const GemmGroups grp, const GemmEpilogue ep) {
   __shared__ float As[kKS][kT + 4], Ws[kKS][kT + 4];
   pdl_launch_dependents();
   pdl_wait();
-  const uint32_t m0 = blockIdx.y * kT, n0 = blockIdx.x * kT;
+  uint32_t m0 = blockIdx.y * kT;
+  const uint32_t n0 = blockIdx.x * kT;
+  if constexpr (GROUPED) {  // blockIdx.y counts the kT-row parts of the group tiles
+    const uint32_t i = blockIdx.y / (kGroupTile / kT);
+    if (i >= *grp.n_tiles) return;
+    const uint2 tile = grp.tiles[i];
+    m0 = tile.y + blockIdx.y % (kGroupTile / kT) * kT;
+    M = grp.rows[tile.x + 1];
+    if (m0 >= M) return;
+    W += (size_t)tile.x * N * K;
+  }
   const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
   float acc[4][4] = {};
   float a_reg[4], w_reg[4];
@@ -71,11 +81,25 @@ cudaError_t launch_gemm_simt(cudaStream_t s, int dtype, const void* A, const voi
                              const GemmEpilogue& ep) {
   if (!A || !W || !M || !N || !K || (ep.kind == GEMM_EPI_GATED && (N & 1u))) return cudaErrorInvalidValue;
   const dim3 grid((N + kT - 1) / kT, (M + kT - 1) / kT);
+  const GemmGroups none;
   if (dtype == 0)
-    return launch_pdl(gemm_simt_kernel<float>, grid, dim3(256), 0, s, prefill_pdl(), (const float*)A, (const float*)W, M, N, K, ep);
+    return launch_pdl(gemm_simt_kernel<float, false>, grid, dim3(256), 0, s, prefill_pdl(), (const float*)A, (const float*)W, M, N, K, none, ep);
   if (dtype == 2)
-    return launch_pdl(gemm_simt_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, prefill_pdl(), (const __nv_bfloat16*)A,
-                      (const __nv_bfloat16*)W, M, N, K, ep);
+    return launch_pdl(gemm_simt_kernel<__nv_bfloat16, false>, grid, dim3(256), 0, s, prefill_pdl(), (const __nv_bfloat16*)A,
+                      (const __nv_bfloat16*)W, M, N, K, none, ep);
+  return cudaErrorInvalidValue;
+}
+
+cudaError_t launch_gemm_simt_grouped(cudaStream_t s, int dtype, const void* A, const void* W, uint32_t N, uint32_t K, const GemmGroups& g,
+                                     const GemmEpilogue& ep) {
+  if (!A || !W || !N || !K || !g.max_tiles || ep.bias || ep.resid || (ep.kind == GEMM_EPI_GATED && (N & 1u))) return cudaErrorInvalidValue;
+  const dim3 grid((N + kT - 1) / kT, g.max_tiles * (kGroupTile / kT));
+  if (grid.y > 65535) return cudaErrorInvalidValue;
+  if (dtype == 0)
+    return launch_pdl(gemm_simt_kernel<float, true>, grid, dim3(256), 0, s, prefill_pdl(), (const float*)A, (const float*)W, 0u, N, K, g, ep);
+  if (dtype == 2)
+    return launch_pdl(gemm_simt_kernel<__nv_bfloat16, true>, grid, dim3(256), 0, s, prefill_pdl(), (const __nv_bfloat16*)A,
+                      (const __nv_bfloat16*)W, 0u, N, K, g, ep);
   return cudaErrorInvalidValue;
 }
 

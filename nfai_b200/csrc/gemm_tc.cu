@@ -292,9 +292,12 @@ __device__ __forceinline__ void bar_arrive(uint32_t bar) {
 // an IEEE division per output) ran at the latency of its dependent instructions and took longer than the tile's MMAs.
 constexpr int kPThreadsGemm = 64 + 8 * 32;
 static_assert(PSmem::kTotal <= 227 * 1024, "shared memory of the persistent kernel");
+// GROUPED: the tiles of rows come from a device list, each with the group whose matrix it is multiplied by; a tile may read
+// rows of A or W beyond its group (they exist or are zero-filled), its epilogue stores the group's own.
+template <bool GROUPED>
 __global__ void __launch_bounds__(kPThreadsGemm) gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap mapA,
-                                                                          const __grid_constant__ CUtensorMap mapW, uint32_t M,
-                                                                          uint32_t N, uint32_t K, const GemmEpilogue ep,
+                                                                          const __grid_constant__ CUtensorMap mapW, const uint32_t M_all,
+                                                                          uint32_t N, uint32_t K, const GemmGroups grp, const GemmEpilogue ep,
                                                                           uint32_t* err) {
   using SM = PSmem;
   constexpr int STAGES = kPStages;
@@ -307,7 +310,8 @@ __global__ void __launch_bounds__(kPThreadsGemm) gemm_tc_persistent_kernel(const
                  tempty0 = s_u32(bars + 2 * STAGES + 2);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const uint32_t KT = (K + kBK - 1) / kBK;
-  const uint32_t mtiles = (M + kBM - 1) / kBM, ntiles = (N + kPBN - 1) / kPBN, tiles = mtiles * ntiles;
+  uint32_t mtiles = (M_all + kBM - 1) / kBM;
+  const uint32_t ntiles = (N + kPBN - 1) / kPBN;
 
   if (threadIdx.x == 0) {
     for (int s = 0; s < STAGES; ++s) {
@@ -332,12 +336,32 @@ __global__ void __launch_bounds__(kPThreadsGemm) gemm_tc_persistent_kernel(const
   // barriers and tensor memory are set up; the operands (and the residual) come from the previous kernel
   pdl_launch_dependents();
   pdl_wait();
+  if constexpr (GROUPED) mtiles = min(*grp.n_tiles, grp.max_tiles);
+  const uint32_t tiles = mtiles * ntiles;
+  struct Tile {
+    uint32_t m0, m_end, n0, w0;  // rows [m0, m_end) of A and the output, columns from n0, rows of W from w0
+  };
+  auto tile_at = [&](uint32_t tile) {
+    Tile t;
+    if constexpr (GROUPED) {  // column tiles fastest: they share the rows of A, which few other tiles do
+      const uint2 g = __ldcg(grp.tiles + tile / ntiles);
+      t.m0 = g.y;
+      t.m_end = __ldcg(grp.rows + g.x + 1);
+      t.n0 = (tile % ntiles) * kPBN;
+      t.w0 = g.x * N + t.n0;
+    } else {
+      t.m0 = (tile % mtiles) * kBM;
+      t.m_end = M_all;
+      t.n0 = t.w0 = (tile / mtiles) * kPBN;
+    }
+    return t;
+  };
 
   if (warp == 0) {
     if (lane == 0) {
       uint32_t it = 0;
       for (uint32_t tile = blockIdx.x; tile < tiles && ok; tile += gridDim.x) {
-        const uint32_t m0 = (tile % mtiles) * kBM, n0 = (tile / mtiles) * kPBN;
+        const Tile at = tile_at(tile);
         for (uint32_t kt = 0; kt < KT; ++kt, ++it) {
           const uint32_t s = it % STAGES;
           if (it >= (uint32_t)STAGES) {
@@ -345,8 +369,8 @@ __global__ void __launch_bounds__(kPThreadsGemm) gemm_tc_persistent_kernel(const
           }
           const uint32_t a_dst = s_u32(gsm + s * SM::kStage), b_dst = a_dst + SM::kABytes;
           bar_expect_tx(full0 + 8 * s, SM::kABytes + SM::kBBytes);
-          tma_load_2d(a_dst, &mapA, (int)(kt * kBK), (int)m0, full0 + 8 * s);
-          tma_load_2d(b_dst, &mapW, (int)(kt * kBK), (int)n0, full0 + 8 * s);
+          tma_load_2d(a_dst, &mapA, (int)(kt * kBK), (int)at.m0, full0 + 8 * s);
+          tma_load_2d(b_dst, &mapW, (int)(kt * kBK), (int)at.w0, full0 + 8 * s);
         }
       }
     }
@@ -380,7 +404,8 @@ __global__ void __launch_bounds__(kPThreadsGemm) gemm_tc_persistent_kernel(const
     uint32_t i = 0;
     for (uint32_t tile = blockIdx.x; tile < tiles; tile += gridDim.x, ++i) {
       const uint32_t acc = i & 1;
-      const uint32_t m0 = (tile % mtiles) * kBM, n0 = (tile / mtiles) * kPBN;
+      const Tile at = tile_at(tile);
+      const uint32_t m0 = at.m0, n0 = at.n0, M = at.m_end;
       // this lane's 16 pairs of a 32 x 32 block: lanes 0-15 along the column pairs of one row, lanes 16-31 on the next
       const uint32_t col = 2u * (lane & 15);
       float* eb = reinterpret_cast<float*>(gsm + SM::kEpiOff) + (warp - 2) * (32 * 33);
@@ -637,22 +662,24 @@ cudaError_t launch_bn(cudaStream_t s, const __half* A, const __half* W, uint32_t
                     (const float*)ep.scratch, M, N, Z, ep);
 }
 
+template <bool GROUPED>
 cudaError_t launch_persistent(cudaStream_t s, const __half* A, const __half* W, uint32_t M, uint32_t N, uint32_t K,
-                              const GemmEpilogue& ep, uint32_t* err) {
+                              const GemmGroups& grp, const GemmEpilogue& ep, uint32_t* err) {
   CUtensorMap mapA, mapW;
-  if (!make_map(&mapA, A, M, K, kBM) || !make_map(&mapW, W, N, K, kPBN)) return cudaErrorInvalidValue;
+  if (!make_map(&mapA, A, M, K, kBM) || !make_map(&mapW, W, GROUPED ? (uint64_t)grp.count * N : N, K, kPBN)) return cudaErrorInvalidValue;
+  auto kern = gemm_tc_persistent_kernel<GROUPED>;
   static thread_local int attr_device = -1;
   int dev = 0;
   cudaError_t e = cudaGetDevice(&dev);
   if (e != cudaSuccess) return e;
   if (attr_device != dev) {
-    e = cudaFuncSetAttribute(gemm_tc_persistent_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)PSmem::kTotal);
+    e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)PSmem::kTotal);
     if (e != cudaSuccess) return e;
     attr_device = dev;
   }
-  const uint32_t tiles = ((M + kBM - 1) / kBM) * ((N + kPBN - 1) / kPBN);
-  return launch_pdl(gemm_tc_persistent_kernel, dim3(tiles < sm_count() ? tiles : sm_count()), dim3(kPThreadsGemm), PSmem::kTotal, s,
-                    prefill_pdl(), mapA, mapW, M, N, K, ep, err);
+  const uint32_t tiles = (GROUPED ? grp.max_tiles : (M + kBM - 1) / kBM) * ((N + kPBN - 1) / kPBN);
+  return launch_pdl(kern, dim3(tiles < sm_count() ? tiles : sm_count()), dim3(kPThreadsGemm), PSmem::kTotal, s, prefill_pdl(), mapA, mapW,
+                    M, N, K, grp, ep, err);
 }
 
 }  // namespace
@@ -678,7 +705,7 @@ cudaError_t launch_gemm_tc(cudaStream_t s, const __half* A, const __half* W, uin
   const uint32_t mtiles = (M + kBM - 1) / kBM;
   // enough 128 x 256 tiles to occupy most SMs: the persistent kernel (NFAI_GEMM_PERSISTENT=0 keeps the tile-per-CTA one)
   static const bool persistent_ok = [] { const char* v = getenv("NFAI_GEMM_PERSISTENT"); return !(v && atoi(v) == 0); }();
-  if (persistent_ok && mtiles * ((N + 255) / 256) >= 96) return launch_persistent(s, A, W, M, N, K, ep, err);
+  if (persistent_ok && mtiles * ((N + 255) / 256) >= 96) return launch_persistent<false>(s, A, W, M, N, K, GemmGroups(), ep, err);
   if (ep.scratch) {
     uint32_t Z = gemm_tc_splits(M, N, K);
     while (Z > 1 && (size_t)Z * M * N > ep.scratch_floats) --Z;
@@ -687,6 +714,14 @@ cudaError_t launch_gemm_tc(cudaStream_t s, const __half* A, const __half* W, uin
   if (mtiles * ((N + 127) / 128) >= 120) return launch_bn<128, 4>(s, A, W, M, N, K, ep, err);
   if (mtiles * ((N + 63) / 64) >= 120) return launch_bn<64, 6>(s, A, W, M, N, K, ep, err);
   return launch_bn<32, 8>(s, A, W, M, N, K, ep, err);
+}
+
+cudaError_t launch_gemm_tc_grouped(cudaStream_t s, const __half* A, const __half* W, uint32_t max_rows, uint32_t N, uint32_t K,
+                                   const GemmGroups& g, const GemmEpilogue& ep, uint32_t* err) {
+  static_assert(kGroupTile == kBM, "the tile list is made for this kernel's tiles");
+  if (!A || !W || !max_rows || !N || !K || (K & 7u) || (((uintptr_t)A | (uintptr_t)W) & 15) || !g.count || !g.max_tiles) return cudaErrorInvalidValue;
+  if (ep.kind == GEMM_EPI_QKV_ROPE || (ep.kind == GEMM_EPI_GATED && (N & 1u)) || ep.bias || ep.resid || ep.operands_bf16 > 1) return cudaErrorInvalidValue;
+  return launch_persistent<true>(s, A, W, max_rows, N, K, g, ep, err);
 }
 
 bool prefill_pdl() {

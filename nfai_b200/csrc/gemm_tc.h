@@ -16,6 +16,9 @@ struct GemmEpilogue {
   void* out_act = nullptr;       // GATED: [M][N/2], STORE_ACT: [M][N], of out_dtype
   int out_dtype = 1;             // 0 float32, 1 float16, 2 bfloat16
   int act = 0;                   // GATED: Activation (kernels.h)
+  float act_limit = 0.f;         // GATED, clamped activation
+  uint32_t gated_cols = 0;       // GATED: only this many columns are gate/up pairs (0: all), the rest go plainly to out_f32
+                                 // [M][N - gated_cols]; even, as is N
   uint32_t operands_bf16 = 0;    // 1: A and W are bfloat16 (both), 0: float16 (both)
   // QKV_ROPE
   void* kcache = nullptr;
@@ -30,6 +33,17 @@ struct GemmEpilogue {
   size_t scratch_floats = 0;
 };
 
+// Rows of A sorted into groups (experts), each multiplied by its own matrix: group g's rows are rows[g] .. rows[g+1]-1 of A
+// and of the output, its matrix is rows g*N .. g*N+N-1 of W. All of it is device data; a kernel walks the tile list.
+struct GemmGroups {
+  uint32_t count = 0;               // number of groups
+  const uint32_t* rows = nullptr;   // [count + 1] first row of each group
+  const uint2* tiles = nullptr;     // (group, first row) of every kGroupTile rows of a group, groups in order
+  const uint32_t* n_tiles = nullptr;
+  uint32_t max_tiles = 0;           // upper bound of *n_tiles
+};
+constexpr uint32_t kGroupTile = 128;
+
 // Number of K splits launch_gemm_tc would use for this shape given enough scratch (1 = no split).
 uint32_t gemm_tc_splits(uint32_t M, uint32_t N, uint32_t K);
 
@@ -37,6 +51,13 @@ uint32_t gemm_tc_splits(uint32_t M, uint32_t N, uint32_t K);
 // err (optional device word) gets bit 4 when a bounded wait inside the kernel gave up.
 cudaError_t launch_gemm_tc(cudaStream_t s, const __half* A, const __half* W, uint32_t M, uint32_t N, uint32_t K,
                            const GemmEpilogue& ep, uint32_t* err);
+
+// The same for grouped rows: A [rows][K] in group order, W [groups][N][K]; epilogues GATED, STORE and STORE_ACT without
+// bias or residual. max_rows bounds the rows of A.
+cudaError_t launch_gemm_tc_grouped(cudaStream_t s, const __half* A, const __half* W, uint32_t max_rows, uint32_t N, uint32_t K,
+                                   const GemmGroups& g, const GemmEpilogue& ep, uint32_t* err);
+cudaError_t launch_gemm_simt_grouped(cudaStream_t s, int dtype, const void* A, const void* W, uint32_t N, uint32_t K, const GemmGroups& g,
+                                     const GemmEpilogue& ep);
 
 // x[M][H] float32 -> RMS-normalised, gain-scaled float16 rows (the A operand of the QKV and gate/up GEMMs).
 // after_collective: x was produced by a library collective enqueued just before; the kernel is then launched with

@@ -26,6 +26,9 @@ using namespace gemv_detail;
 // gemv_bf16.cu
 cudaError_t launch_gemv_more(int wdtype, GemvEpilogue epi, bool vec, int R, int U, dim3 grid, size_t smem, cudaStream_t s,
                              bool pdl, const GemvParams& p);
+// gemv_moe.cu
+cudaError_t launch_gemv_experts(int wdtype, GemvEpilogue epi, bool vec, int R, int U, dim3 grid, size_t smem, cudaStream_t s,
+                                bool pdl, const GemvParams& p);
 
 namespace {
 
@@ -54,6 +57,7 @@ cudaError_t launch_e(GemvEpilogue epi, bool vec, int R, int U, dim3 grid, size_t
 
 bool vector_ok(int wdtype, const GemvParams& p) {
   const uint32_t ve = wdtype == 0 ? 4 : 8;
+  if (p.map == MAP_EXPERT_COLUMNS && (p.expert.seg % ve != 0 || (reinterpret_cast<uintptr_t>(p.expert.W2) & 15) != 0)) return false;
   return p.K % ve == 0 && (reinterpret_cast<uintptr_t>(p.W) & 15) == 0;
 }
 
@@ -68,7 +72,7 @@ int rows_per_warp(GemvEpilogue epi, bool vec, const GemvTune& t) {
 
 static bool use_ring(int wdtype, GemvEpilogue epi, const GemvParams& p, const GemvTune& t) {
   if (t.mode != 1 || !vector_ok(wdtype, p)) return false;
-  if (wdtype == 2 || epi == EPI_HYPER || p.norm_groups > 1 || p.y_ring) return false;
+  if (wdtype == 2 || epi == EPI_HYPER || p.norm_groups > 1 || p.y_ring || p.post.y || p.map || p.gated_rows) return false;
   return t.unroll >= 1 && t.unroll <= 4 && gemv_ring_smem(p, t.unroll) <= 227 * 1024;
 }
 
@@ -131,8 +135,19 @@ cudaError_t launch_gemv(cudaStream_t s, int wdtype, int kvdtype, GemvEpilogue ep
   dim3 grid(gemv_grid(wdtype, epi, p, t));
   p.split_log2 = gemv_split_log2(wdtype, vec, R, p, t);
   if (p.norm_groups > 1 && (!p.gain || p.K % p.norm_groups)) return cudaErrorInvalidValue;
-  size_t smem = (kSmemHeader + (size_t)p.K * (p.gain ? 2 : 1)) * sizeof(float);
+  if (p.gated_rows && (epi != EPI_GATED || !p.tail || (p.gated_rows & 1u))) return cudaErrorInvalidValue;
+  if (p.post.y && (!p.post.gain || p.tp.pull || p.norm_groups > 1)) return cudaErrorInvalidValue;
+  size_t smem = (kSmemHeader + (size_t)gemv_x_floats(p) + gemv_map_floats(p, wdtype == 0 ? 4 : 8)) * sizeof(float);
   if (smem > 227 * 1024) return cudaErrorInvalidValue;
+  if (p.map) {
+    const ExpertMap& x = p.expert;
+    if (p.map == MAP_EXPERT_ROWS && (epi != EPI_GATED || !x.rows || (x.rows & 1u) || p.N != x.router.top * x.rows || !x.logits || !x.chosen ||
+                                     x.router.top > 32 || x.router.experts > kMaxExperts || x.router.groups > kMaxGroups))
+      return cudaErrorInvalidValue;
+    if (p.map == MAP_EXPERT_COLUMNS && (epi != EPI_STORE || !x.seg || !x.chosen || p.K < x.top * x.seg || (p.K > x.top * x.seg && (!x.W2 || !x.shared_gate))))
+      return cudaErrorInvalidValue;
+    return launch_gemv_experts(wdtype, epi, vec, R, t.unroll, grid, smem, s, pdl, p);
+  }
   if (wdtype == 2 || epi == EPI_HYPER) {
     if (epi == EPI_QKV_ROPE || (epi == EPI_HYPER && (!p.hyper.S || p.hyper.S > kMaxStreams))) return cudaErrorInvalidValue;
     return launch_gemv_more(wdtype, epi, vec, R, t.unroll, grid, smem, s, pdl, p);

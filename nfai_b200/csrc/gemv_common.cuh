@@ -14,7 +14,7 @@ constexpr int kWarps = kThreads / 32;
 __device__ __forceinline__ void load_gain(const GemvParams& p, float* xs, float* gs_at = nullptr) {
   if (p.gain == nullptr) return;
   float* gs = gs_at ? gs_at : xs + p.K;
-  for (uint32_t i = threadIdx.x; i < p.K; i += kThreads) gs[i] = p.gain[i];
+  for (uint32_t i = threadIdx.x; i < p.K; i += kThreads) gs[i] = p.gain[i * p.gain_stride];
 }
 
 // Tensor-parallel input: x = residual + the partial vectors of all ranks, which the previous row-parallel GEMV of
@@ -81,6 +81,70 @@ __device__ __forceinline__ uint32_t x_slot4(uint32_t i4) {  // index of the floa
 template <bool PERM>
 __device__ __forceinline__ uint32_t x_slot(uint32_t k) { return 4u * x_slot4<PERM>(k >> 2) + (k & 3u); }
 
+// Sum over the CTA, the same on every thread; `red` holds kWarps floats and may be reused right after.
+__device__ __forceinline__ float cta_sum(float v, float* red) {
+  v = warp_sum(v);
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+  __syncthreads();
+  float tot = 0.f;
+#pragma unroll
+  for (int w = 0; w < kWarps; ++w) tot += red[w];
+  __syncthreads();
+  return tot;
+}
+
+// x = base + mult * gain * (y / rms(y)) into xs (PostNorm); `bs` has room for K more floats. Returns this thread's share of
+// the sum of squares of x. Both vectors are requested before either is used.
+__device__ __forceinline__ float load_post_norm(const GemvParams& p, float* xs, float* bs, float* red) {
+  const uint32_t K = p.K, tid = threadIdx.x;
+  const PostNorm& t = p.post;
+  const bool quads = (K & 3u) == 0 && ((reinterpret_cast<uintptr_t>(p.x) | reinterpret_cast<uintptr_t>(t.y)) & 15) == 0;
+  const float c = t.mult * __ldg(t.gain);
+  float ss = 0.f;
+  if (quads) {
+    const uint32_t n4 = K >> 2;
+    constexpr int B = 4;
+    for (uint32_t base = 0; base < n4; base += B * kThreads) {
+      float4 y[B], b[B];
+#pragma unroll
+      for (int j = 0; j < B; ++j) {
+        const uint32_t i = base + j * kThreads + tid;
+        y[j] = i < n4 ? __ldcg(reinterpret_cast<const float4*>(t.y) + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        b[j] = i < n4 ? __ldcg(reinterpret_cast<const float4*>(p.x) + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+      }
+#pragma unroll
+      for (int j = 0; j < B; ++j) {
+        const uint32_t i = base + j * kThreads + tid;
+        if (i < n4) {
+          reinterpret_cast<float4*>(xs)[i] = y[j];
+          reinterpret_cast<float4*>(bs)[i] = b[j];
+          ss = fmaf(y[j].x, y[j].x, ss);
+          ss = fmaf(y[j].y, y[j].y, ss);
+          ss = fmaf(y[j].z, y[j].z, ss);
+          ss = fmaf(y[j].w, y[j].w, ss);
+        }
+      }
+    }
+  } else {
+    for (uint32_t i = tid; i < K; i += kThreads) {
+      const float v = __ldcg(t.y + i);
+      xs[i] = v;
+      bs[i] = __ldcg(p.x + i);
+      ss = fmaf(v, v, ss);
+    }
+  }
+  const float rms = sqrtf(__fdiv_rn(cta_sum(ss, red), (float)K) + t.eps);
+  const bool keep = blockIdx.x == 0 && t.store;
+  float sx = 0.f;
+  for (uint32_t i = tid; i < K; i += kThreads) {
+    const float v = fmaf(c, __fdiv_rn(xs[i], rms), bs[i]);
+    xs[i] = v;
+    if (keep) t.store[i] = v;
+    sx = fmaf(v, v, sx);
+  }
+  return sx;
+}
+
 // ss = sum x^2 ; rms = sqrt(ss/K + eps) ; xs = (x / rms) * gain   (RMSNormShader.cs:136-148)
 // With PERM the shared-memory area of x must be a whole number of 256-element blocks.
 template <bool PERM = false>
@@ -93,7 +157,9 @@ __device__ __forceinline__ void load_x(const GemvParams& p, float* xs, float* re
   const float* gs = gs_in ? gs_in : xs + K;  // staged by load_gain() before the dependency wait
   const bool norm = p.gain != nullptr;
   float ss = 0.f;
-  if (pull) {  // the host guarantees K % 4 == 0 and 16-byte aligned vectors for a pulling kernel
+  if (!PERM && p.post.y) {
+    ss = load_post_norm(p, xs, xs + (norm ? 2 : 1) * K, red);
+  } else if (pull) {  // the host guarantees K % 4 == 0 and 16-byte aligned vectors for a pulling kernel
     const uint32_t pull_epoch = *p.tp.epoch_base + p.tp.pull_index + 1;
     bool pull_ok = true;
     for (uint32_t i = tid; i < (K >> 2); i += kThreads) {
@@ -261,7 +327,12 @@ __device__ __forceinline__ void row_epilogue(const GemvParams& p, uint32_t row0,
       if (n >= p.N) break;
       // sigmoid = 1/(1+exp(-x)); silu = x*sigmoid; h = up*silu (SiLUShader.cs:121-123, ElementWiseMul A=up,B=silu)
       const float gate = p.bias ? acc[r] + __ldg(p.bias + n) : acc[r], up = p.bias ? acc[r + 1] + __ldg(p.bias + n + 1) : acc[r + 1];
-      p.y[n >> 1] = gated(p.act, gate, up);
+      if (p.gated_rows && n >= p.gated_rows) {  // (n is even, and so is gated_rows)
+        p.tail[n - p.gated_rows] = acc[r];
+        if (n + 1 < p.N) p.tail[n + 1 - p.gated_rows] = acc[r + 1];
+        continue;
+      }
+      p.y[n >> 1] = gated(p.act, gate, up, p.act_limit);
     }
   } else {  // EPI_LOGITS: store and keep the warp's best (lowest index among equal maxima)
 #pragma unroll
@@ -317,7 +388,7 @@ __device__ __forceinline__ void epi_preload(const GemvParams& p, uint32_t row0, 
   }
 }
 
-template <typename KVT, int R, int EPI>
+template <typename KVT, int R, int EPI, int MAP = MAP_PLAIN>
 __device__ __forceinline__ void row_epilogue_pre(const GemvParams& p, uint32_t row0, const float (&acc)[R],
                                                  const float (&pre)[R], uint32_t pos, float& best_v, uint32_t& best_i) {
   if constexpr (EPI == EPI_HYPER) {  // the whole warp: lane t makes stream t
@@ -346,6 +417,13 @@ __device__ __forceinline__ void row_epilogue_pre(const GemvParams& p, uint32_t r
     return;
   }
   if ((threadIdx.x & 31) != 0) return;
+  if constexpr (MAP == MAP_EXPERT_ROWS) {  // `pre` holds the weights of the rows' experts
+    static_assert(EPI == EPI_GATED && R % 2 == 0, "gate and up rows are interleaved");
+#pragma unroll
+    for (int r = 0; r < R; r += 2)
+      if (row0 + r < p.N) p.y[(row0 + r) >> 1] = pre[r] * gated(p.act, acc[r], acc[r + 1], p.act_limit);
+    return;
+  }
   if constexpr (EPI == EPI_STORE) {
     if (p.tp.push) {
       push_rows<R>(p, row0, acc);

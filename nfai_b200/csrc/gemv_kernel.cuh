@@ -1,6 +1,7 @@
 // The register-streaming GEMV kernel (see gemv.cu for its design) and its launch helpers, as templates.
 #pragma once
 #include "gemv_common.cuh"
+#include "moe_route.cuh"
 
 namespace nfai {
 
@@ -10,8 +11,58 @@ namespace {  // every including translation unit instantiates its own combinatio
 
 constexpr int kSmemHeader = 96;  // floats ahead of x in shared memory: reduction scratch and split-row partials
 
+// ---- weights found through the chosen experts (WeightMap) ----------------------------------------------------------
+// Shared memory behind x, the gain and the base of a post-norm residual.
+__host__ __device__ inline uint32_t gemv_x_floats(const GemvParams& p) {
+  return (p.K * (1u + (p.gain ? 1u : 0u) + (p.post.y ? 1u : 0u)) + 3u) & ~3u;
+}
+__host__ __device__ inline uint32_t gemv_map_floats(const GemvParams& p, uint32_t vec_elems) {
+  if (p.map == MAP_EXPERT_ROWS) return 2 * kMaxChosen + kRouteScratch + p.expert.router.experts;
+  if (p.map == MAP_EXPERT_COLUMNS) return 2 * (p.K / vec_elems);  // one pointer per vector of a row
+  return 0;
+}
+struct ChosenRows {  // MAP_EXPERT_ROWS
+  const uint32_t* ids;
+  const float* w;
+  __device__ __forceinline__ ChosenRows(const GemvParams& p, float* area) : ids(reinterpret_cast<uint32_t*>(area)), w(area + kMaxChosen) {}
+  // warp 0 chooses, CTA 0 keeps the choice for the product that follows
+  __device__ __forceinline__ static void choose(const GemvParams& p, float* area) {
+    if (threadIdx.x < 32) {
+      uint32_t* const ids = reinterpret_cast<uint32_t*>(area);
+      route_warp(p.expert.router, p.expert.logits, area + 2 * kMaxChosen + kRouteScratch, area + 2 * kMaxChosen, ids, area + kMaxChosen);
+      if (blockIdx.x == 0 && threadIdx.x < p.expert.router.top) p.expert.chosen[threadIdx.x] = ids[threadIdx.x];
+    }
+    __syncthreads();
+  }
+  __device__ __forceinline__ size_t row(const GemvParams& p, uint32_t n) const {  // row of W
+    const uint32_t k = n / p.expert.rows;
+    return (size_t)ids[k] * p.expert.rows + (n - k * p.expert.rows);
+  }
+};
+// MAP_EXPERT_COLUMNS: element k of row 0; the rows of its matrix are *ld elements apart
+template <typename WT>
+__device__ __forceinline__ const WT* chosen_column(const GemvParams& p, uint32_t k, uint32_t* ld) {
+  const ExpertMap& m = p.expert;
+  const uint32_t split = m.top * m.seg;
+  if (k >= split) {
+    *ld = p.K - split;
+    return reinterpret_cast<const WT*>(m.W2) + (k - split);
+  }
+  const uint32_t i = k / m.seg;
+  *ld = m.seg;
+  return reinterpret_cast<const WT*>(p.W) + (size_t)__ldcg(m.chosen + i) * p.N * m.seg + (k - i * m.seg);
+}
+// x behind the experts' parts belongs to the shared feed-forward
+__device__ __forceinline__ void scale_shared(const GemvParams& p, float* xs) {
+  const uint32_t split = p.expert.top * p.expert.seg;
+  if (split >= p.K) return;
+  const float g = route_sigmoid(__ldcg(p.expert.shared_gate));
+  for (uint32_t i = split + threadIdx.x; i < p.K; i += kThreads) xs[i] *= g;
+  __syncthreads();
+}
+
 // ---- the streamer ---------------------------------------------------------------------------------------------
-template <typename WT, typename KVT, int R, int U, int EPI>
+template <typename WT, typename KVT, int R, int U, int EPI, int MAP = MAP_PLAIN>
 __global__ void __launch_bounds__(kThreads, 2) gemv_kernel(const GemvParams p) {
   extern __shared__ __align__(16) float smem[];
   float* red = smem;                  // 2*kWarps words of reduction scratch
@@ -30,21 +81,40 @@ __global__ void __launch_bounds__(kThreads, 2) gemv_kernel(const GemvParams p) {
   const uint32_t nrounds = (nitems + TW - 1) / TW;  // the same for every warp of the grid: barriers stay uniform
   const WT* const Wbase = reinterpret_cast<const WT*>(p.W);
   const uint4 zero = make_uint4(0, 0, 0, 0);
+  float* const area = xs + gemv_x_floats(p);
+  const ChosenRows rows(p, area);                           // MAP_EXPERT_ROWS
+  const WT** const cols = reinterpret_cast<const WT**>(area);  // MAP_EXPERT_COLUMNS: vector v of row 0
+  const uint32_t cols_split = MAP == MAP_EXPERT_COLUMNS ? p.expert.top * p.expert.seg / VE : 0u;
 
   auto load_batch = [&](uint4(&buf)[U][R], uint32_t t, uint32_t kb) {
     if (t >= nitems) return;
     const uint32_t rb = t >> sl, c = t & (S - 1);
     const uint32_t v0 = c * cv + kb * (32 * U) + lane;
     const uint32_t vend = min((c + 1) * cv, nvec);
-#pragma unroll
-    for (int r = 0; r < R; ++r) {
-      uint32_t n = rb * R + r;
-      n = n < p.N ? n : p.N - 1;  // a ragged last block re-reads the last row, never out of bounds
-      const uint4* wrow = reinterpret_cast<const uint4*>(Wbase + (size_t)n * p.K);
+    if constexpr (MAP == MAP_EXPERT_COLUMNS) {
 #pragma unroll
       for (int u = 0; u < U; ++u) {
         const uint32_t v = v0 + 32 * u;
-        buf[u][r] = v < vend ? ld_stream16(wrow + v) : zero;
+        const WT* col = v < vend ? cols[v] : nullptr;
+        const uint32_t ld = v < cols_split ? p.expert.seg : p.K - p.expert.top * p.expert.seg;
+#pragma unroll
+        for (int r = 0; r < R; ++r) {
+          uint32_t n = rb * R + r;
+          n = n < p.N ? n : p.N - 1;
+          buf[u][r] = v < vend ? ld_stream16(col + (size_t)n * ld) : zero;
+        }
+      }
+    } else {
+#pragma unroll
+      for (int r = 0; r < R; ++r) {
+        uint32_t n = rb * R + r;
+        n = n < p.N ? n : p.N - 1;  // a ragged last block re-reads the last row, never out of bounds
+        const uint4* wrow = reinterpret_cast<const uint4*>(Wbase + (MAP == MAP_EXPERT_ROWS ? rows.row(p, n) : (size_t)n) * p.K);
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+          const uint32_t v = v0 + 32 * u;
+          buf[u][r] = v < vend ? ld_stream16(wrow + v) : zero;
+        }
       }
     }
   };
@@ -60,18 +130,34 @@ __global__ void __launch_bounds__(kThreads, 2) gemv_kernel(const GemvParams p) {
   // Weights do not depend on the previous kernel: the first batch is requested before the dependency wait.
   // (Requesting the first two there, in either loop order, measured 10-30% slower in the steady state.)
   uint4 cur[U][R], nxt[U][R];
-  load_batch(cur, lt, lkb);
-  advance();
+  if constexpr (MAP == MAP_PLAIN) {
+    load_batch(cur, lt, lkb);
+    advance();
+  }
   load_gain(p, xs);
   prefetch_plan(p.pf, kPrefetchChunk);
   pdl_launch_dependents();
   pdl_wait();
+  if constexpr (MAP != MAP_PLAIN) {  // which weights are needed is part of the previous kernel's result
+    if constexpr (MAP == MAP_EXPERT_ROWS) {
+      ChosenRows::choose(p, area);
+    } else {
+      for (uint32_t v = threadIdx.x; v < nvec; v += kThreads) {
+        uint32_t ld;
+        cols[v] = chosen_column<WT>(p, v * VE, &ld);
+      }
+      __syncthreads();
+    }
+    load_batch(cur, lt, lkb);
+    advance();
+  }
   // what the epilogue of the first item reads (residual / cos, sin of this position) travels with x
   uint32_t pos = 0;
   if (EPI == EPI_QKV_ROPE || (EPI == EPI_STORE && p.y_ring)) pos = p.state ? p.state->pos : p.pos_imm;
   float pre[R];
   epi_preload<R, EPI>(p, (min(t, nitems - 1) >> sl) * R, pos, pre);
   load_x(p, xs, red);
+  if constexpr (MAP == MAP_EXPERT_COLUMNS) scale_shared(p, xs);
 
   float best_v = -INFINITY;
   uint32_t best_i = 0xffffffffu;
@@ -117,11 +203,15 @@ __global__ void __launch_bounds__(kThreads, 2) gemv_kernel(const GemvParams p) {
 #pragma unroll
         for (int r = 0; r < R; ++r) cur[u][r] = nxt[u][r];
     }
+    if constexpr (MAP == MAP_EXPERT_ROWS) {  // the weight of the pair's expert takes the place of what an epilogue preloads
+#pragma unroll
+      for (int r = 0; r < R; ++r) pre[r] = rows.w[min((t >> sl) * R + r, p.N - 1) / p.expert.rows];
+    }
     // the item is complete
 #pragma unroll
     for (int r = 0; r < R; ++r) acc[r] = warp_sum(acc[r]);
     if (S == 1) {
-      if (t < nitems) row_epilogue_pre<KVT, R, EPI>(p, t * R, acc, pre, pos, best_v, best_i);
+      if (t < nitems) row_epilogue_pre<KVT, R, EPI, MAP>(p, t * R, acc, pre, pos, best_v, best_i);
     } else {
       // the S chunks of a row block sit in S consecutive warps of this CTA: add them up in warp order
       float* pr = part + (round & 1) * (kWarps * R);
@@ -137,7 +227,7 @@ __global__ void __launch_bounds__(kThreads, 2) gemv_kernel(const GemvParams p) {
           for (uint32_t j = 1; j < S; ++j) a += pr[(warp + j) * R + r];
           acc[r] = a;
         }
-        row_epilogue_pre<KVT, R, EPI>(p, (t >> sl) * R, acc, pre, pos, best_v, best_i);
+        row_epilogue_pre<KVT, R, EPI, MAP>(p, (t >> sl) * R, acc, pre, pos, best_v, best_i);
       }
     }
 #pragma unroll
@@ -150,7 +240,7 @@ __global__ void __launch_bounds__(kThreads, 2) gemv_kernel(const GemvParams p) {
 }
 
 // Same contract for any K and any alignment (element loads); used when K is not a multiple of the vector width.
-template <typename WT, typename KVT, int EPI>
+template <typename WT, typename KVT, int EPI, int MAP = MAP_PLAIN>
 __global__ void __launch_bounds__(kThreads) gemv_scalar_kernel(const GemvParams p) {
   extern __shared__ __align__(16) float smem[];
   float* red = smem;
@@ -163,7 +253,11 @@ __global__ void __launch_bounds__(kThreads) gemv_scalar_kernel(const GemvParams 
   pdl_launch_dependents();
   pdl_wait();
   const uint32_t pos = EPI == EPI_STORE && p.y_ring ? (p.state ? p.state->pos : p.pos_imm) : 0u;
+  float* const area = xs + gemv_x_floats(p);
+  const ChosenRows rows(p, area);
+  if constexpr (MAP == MAP_EXPERT_ROWS) ChosenRows::choose(p, area);
   load_x(p, xs, red);
+  if constexpr (MAP == MAP_EXPERT_COLUMNS) scale_shared(p, xs);
   float best_v = -INFINITY;
   uint32_t best_i = 0xffffffffu;
   for (uint32_t rb = blockIdx.x * kWarps + warp; rb < nrb; rb += gridDim.x * kWarps) {
@@ -171,15 +265,28 @@ __global__ void __launch_bounds__(kThreads) gemv_scalar_kernel(const GemvParams 
 #pragma unroll
     for (int r = 0; r < R; ++r) {
       uint32_t n = rb * R + r < p.N ? rb * R + r : p.N - 1;
-      const WT* w = reinterpret_cast<const WT*>(p.W) + (size_t)n * p.K;
       float a = 0.f;
-      for (uint32_t k = lane; k < p.K; k += 32) a = fmaf(to_float(w[k]), xs[k], a);
+      if constexpr (MAP == MAP_EXPERT_COLUMNS) {
+        for (uint32_t k = lane; k < p.K; k += 32) {
+          uint32_t ld;
+          const WT* col = chosen_column<WT>(p, k, &ld);
+          a = fmaf(to_float(col[(size_t)n * ld]), xs[k], a);
+        }
+      } else {
+        const WT* w = reinterpret_cast<const WT*>(p.W) + (MAP == MAP_EXPERT_ROWS ? rows.row(p, n) : (size_t)n) * p.K;
+        for (uint32_t k = lane; k < p.K; k += 32) a = fmaf(to_float(w[k]), xs[k], a);
+      }
       acc[r] = warp_sum(a);
     }
-    if constexpr (EPI == EPI_STORE || EPI == EPI_HYPER) {
+    if constexpr (EPI == EPI_STORE || EPI == EPI_HYPER || MAP == MAP_EXPERT_ROWS) {
       float pre[R];
-      epi_preload<R, EPI>(p, rb * R, pos, pre);
-      row_epilogue_pre<KVT, R, EPI>(p, rb * R, acc, pre, pos, best_v, best_i);
+      if constexpr (MAP == MAP_EXPERT_ROWS) {
+#pragma unroll
+        for (int r = 0; r < R; ++r) pre[r] = rows.w[rb * R / p.expert.rows];  // (both rows of a pair: one expert)
+      } else {
+        epi_preload<R, EPI>(p, rb * R, pos, pre);
+      }
+      row_epilogue_pre<KVT, R, EPI, MAP>(p, rb * R, acc, pre, pos, best_v, best_i);
     } else {
       row_epilogue<KVT, R, EPI>(p, rb * R, acc, best_v, best_i);
     }

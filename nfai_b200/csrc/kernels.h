@@ -86,13 +86,13 @@ constexpr uint32_t kPrefetchChunk = 4096;
 enum GemvEpilogue {
   EPI_STORE = 0,     // y = acc (+ resid)
   EPI_QKV_ROPE = 1,  // rows are [Q | K | V]; RoPE on Q and K; K,V rows go to the cache at row pos
-  EPI_GATED = 2,     // rows are interleaved (gate_j, up_j); h_j = up_j * act(gate_j)
+  EPI_GATED = 2,     // rows are interleaved (gate_j, up_j); h_j = up_j * act(gate_j); rows from gated_rows on are stored plainly
   EPI_LOGITS = 3,    // y = acc and a per-CTA (max, lowest index) partial
   EPI_HYPER = 4      // y = acc is written into all residual streams (hyper-connections, see HyperWrite)
 };
 
 // Activation of a gated feed-forward.
-enum Activation { ACT_SILU = 0, ACT_RELU = 1 };
+enum Activation { ACT_SILU = 0, ACT_RELU = 1, ACT_CLAMPED = 2 };
 
 // Hyper-connections: the residual is kept as S streams x_s. A sublayer reads u = sum_s in[s] x_s and its output y is
 // written back into all of them: x'_t = sum_s mix[s][t] x_s + out[t] y. The kernel that writes also forms what the NEXT
@@ -107,6 +107,38 @@ struct HyperWrite {
   uint32_t S = 0;                  // <= kMaxStreams
 };
 constexpr uint32_t kMaxStreams = 16;
+
+// A residual that takes the normed output of the previous sublayer: the reader forms x = base + mult * gain * y / rms(y)
+// itself, and its first CTA keeps the result. y null: nothing to add.
+struct PostNorm {
+  const float* y = nullptr;     // [K]
+  const float* gain = nullptr;  // one number
+  float mult = 0.f, eps = 0.f;
+  float* store = nullptr;       // [K]
+};
+
+// Choice of experts from router logits (moe_route.cuh).
+struct Router {
+  const float* correction = nullptr;  // [experts] added to the scores for the choice only
+  uint32_t experts = 0, top = 0, groups = 1, keep = 1;
+  float scale = 1.f;
+};
+
+// How a GEMV finds its weights when the chosen experts decide.
+//   MAP_EXPERT_ROWS    W is [experts][rows][K]; row n of the product is row n % rows of the (n / rows)-th chosen expert, its
+//                      gated output times that expert's weight. Every CTA works the choice out for itself; CTA 0 keeps it.
+//   MAP_EXPERT_COLUMNS the product over K = [top x seg | shared]: part k of x meets row n of W + chosen[k] * N * seg, the last
+//                      part meets W2 and is first multiplied by the sigmoid of *shared_gate.
+enum WeightMap { MAP_PLAIN = 0, MAP_EXPERT_ROWS = 1, MAP_EXPERT_COLUMNS = 2 };
+struct ExpertMap {
+  Router router;
+  const float* logits = nullptr;  // MAP_EXPERT_ROWS
+  uint32_t rows = 0;              // MAP_EXPERT_ROWS: rows per expert (even)
+  uint32_t* chosen = nullptr;     // [top], written / read
+  uint32_t seg = 0, top = 0;      // MAP_EXPERT_COLUMNS
+  const void* W2 = nullptr;       // [N][K - top*seg]
+  const float* shared_gate = nullptr;
+};
 
 struct GemvParams {
   const void* W = nullptr;  // [N][K] row-major, float or half
@@ -144,6 +176,13 @@ struct GemvParams {
   // EPI_STORE into a ring of rows: y is row (position % y_ring) of a buffer of rows y_stride floats apart (0 = plain y)
   uint32_t y_ring = 0, y_stride = 0;
   HyperWrite hyper;             // EPI_HYPER
+  float act_limit = 0.f;        // EPI_GATED, clamped activation
+  uint32_t gain_stride = 1;     // 0: gain is one number for all of x
+  PostNorm post;
+  uint32_t gated_rows = 0;      // EPI_GATED: rows from here on are stored plainly to tail (even; 0: none)
+  float* tail = nullptr;
+  int map = MAP_PLAIN;
+  ExpertMap expert;
 };
 
 // Tunable launch shape of the GEMV family.

@@ -185,7 +185,8 @@ cudaError_t plan_record_step(nfai_model* m, bool with_head, bool from_prompt, in
 int plan_prefill(nfai_model* m, const uint32_t* tokens, int n, const uint32_t* want, int n_want, float* logits_out);
 bool plan_batched(const nfai_model* m);
 int plan_step_launches(const nfai_model* m);
-GemvParams plan_head_params(nfai_model* m);
+// settled: the residual behind the last layer is already in place (a prompt pass leaves it there)
+GemvParams plan_head_params(nfai_model* m, bool settled = false);
 size_t plan_snapshot_bytes(const nfai_model* m, uint32_t pos);
 cudaError_t plan_snapshot_copy(nfai_model* m, uint32_t pos, char* buf, bool save);
 int plan_read_kv(nfai_model* m, uint32_t layer, uint32_t pos, float* k, float* v);

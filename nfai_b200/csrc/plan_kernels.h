@@ -4,6 +4,9 @@
 #include <cuda_runtime.h>
 #include <stdint.h>
 
+#include <string>
+
+#include "gemm_tc.h"
 #include "kernels.h"
 #include "plan.h"
 
@@ -99,5 +102,86 @@ size_t ssm_chunk_floats(const SsmSpec& s, uint32_t T);
 // out[t] = RMS norm of y[t] in `groups` equal parts, times gain, as out_dtype.
 cudaError_t launch_group_norm_rows(cudaStream_t s, const float* y, const float* gain, float eps, uint32_t groups, uint32_t T,
                                    uint32_t K, void* out, int out_dtype);
+
+// ---- residual with post-norms over rows of tokens (post_rows.cu) -----------------------------------------------------
+// One row (token) per CTA: x = base + mult * gain * (y / rms(y)); the row itself, or its RMS norm, is the next operand.
+//   base   embedding row of tokens[row] plus the position vector of pos0 + row, or row rows[i] (default i) of X
+//   y      a sublayer's rows, or the weighted sum of expert rows and a gated shared row (moe_top > 0); null: x = base
+struct PostRows {
+  const uint32_t* tokens = nullptr;
+  const void* embed = nullptr;        // [V][H] of embed_dtype
+  int embed_dtype = 0;
+  const double* freq = nullptr;       // [(H+1)/2] angles per position of the position vector; null: none
+  uint32_t pos0 = 0;
+  const float* X = nullptr;           // [..][H]
+  const uint32_t* rows = nullptr;
+  const float* y = nullptr;           // [T][H]; with moe_top: the shared feed-forward's rows (may be null)
+  uint32_t moe_top = 0;
+  const float* ye = nullptr;          // expert rows [T*top][H]
+  const uint32_t* where = nullptr;    // [T][top] rows of ye
+  const float* w = nullptr;           // [T][top]
+  const float* shared_gate = nullptr; // its sigmoid scales row t of y; shared_ld floats apart
+  uint32_t shared_ld = 0;
+  const float* gain = nullptr;        // one number
+  float mult = 0.f, eps = 0.f;
+  float* X_out = nullptr;             // [T][H]
+  void* operand = nullptr;            // [T][H] of operand_dtype
+  int operand_dtype = 0;
+  const float* norm_gain = nullptr;   // one number: the operand is x / rms(x) * norm_gain
+  float* tap = nullptr;               // [H] copy of row tap_row of x
+  uint32_t tap_row = 0;
+  uint32_t H = 0;
+};
+cudaError_t launch_post_rows(cudaStream_t s, const PostRows& p, uint32_t n_rows);
+// Decode step: embedding plus position vector of the token in *state (its prompt buffer if given).
+cudaError_t launch_embed_position(cudaStream_t s, int wdtype, const void* E, uint32_t H, uint32_t V, StepState* state,
+                                  const uint32_t* prompt, const double* freq, float* x, bool pdl);
+
+// ---- grouped-query attention with head norms, distance bias and head gates (gqa_decode.cu, gqa_prefill.cu) ---------------
+struct GqaParams {
+  GqaSpec spec;
+  const float* in = nullptr;   // projected rows [q | k | v | gate], in_ld floats apart
+  uint32_t in_ld = 0;
+  float eps = 0.f;
+  void* k_cache = nullptr;     // [ctx][kv_heads*dim] of dtype, normed
+  void* v_cache = nullptr;     // [ctx][kv_heads*vdim] of dtype, normed
+  int dtype = 0;               // of caches and operands: 0 or 2
+  uint32_t ctx = 0;
+  StepState* state = nullptr;  // decode: position
+  uint32_t pos0 = 0;           // prompt path: position of the first token
+  // decode
+  float* out = nullptr;        // [heads*vdim], gated
+  float* part = nullptr;       // gqa_decode_scratch bytes, zero-filled once (split partials, then tickets)
+  // prompt path
+  void* q = nullptr;           // [T][heads*dim] of dtype, normed, times scale * log2(e)
+  void* ao = nullptr;          // [T][heads*vdim] of dtype, gated
+};
+bool gqa_supported(const GqaSpec& s, std::string* why);
+size_t gqa_decode_scratch(const GqaSpec& s, uint32_t ctx);
+// Rows of one KV head's keys a decode step at position `pos` has to read, summed over the KV heads.
+uint64_t gqa_rows_read(const GqaSpec& s, uint32_t pos);
+cudaError_t launch_gqa_decode(cudaStream_t s, const GqaParams& p, bool pdl);
+// Norm what the projection of T tokens left: cache rows pos0 .. pos0+T-1 (unless borrowed) and p.q.
+cudaError_t launch_gqa_prep(cudaStream_t s, const GqaParams& p, uint32_t T);
+cudaError_t launch_gqa_prefill(cudaStream_t s, const GqaParams& p, uint32_t T);
+
+// ---- routed feed-forwards over rows of tokens (moe.cu) -------------------------------------------------------------------
+struct MoeRows {
+  Router router;
+  const float* logits = nullptr;  // [T][ld]
+  uint32_t ld = 0;
+  uint32_t* ids = nullptr;        // [T][top]
+  float* w = nullptr;             // [T][top]
+  uint32_t* where = nullptr;      // [T][top] row of the sorted order
+  uint32_t* src = nullptr;        // [T*top] token of a sorted row
+  uint32_t* rows = nullptr;       // [experts + 1]
+  uint2* tiles = nullptr;         // moe_max_tiles entries
+  uint32_t* n_tiles = nullptr;
+};
+uint32_t moe_max_tiles(const MoeSpec& s, uint32_t T);
+// Choose experts for T tokens and sort the (token, choice) pairs by expert, tokens in order.
+cudaError_t launch_moe_route(cudaStream_t s, const MoeRows& p, uint32_t T);
+// out[i] = A[src[i]]: operand rows of H elements (elem bytes each) in sorted order.
+cudaError_t launch_moe_gather(cudaStream_t s, const void* A, const uint32_t* src, uint32_t n, uint32_t H, uint32_t elem, void* out);
 
 }  // namespace nfai

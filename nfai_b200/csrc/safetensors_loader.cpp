@@ -116,7 +116,8 @@ extern "C" int nfai_model_load_dir(nfai_ctx* c, const char* dir, uint32_t kv_cac
   nfai_model* m = nullptr;
   int rc = nfai_model_create_from_config(c, cfg.p, cfg.n, kv_cache_size, weight_dtype, &m);
   for (size_t i = 0; rc == NFAI_OK && i < need.size(); ++i) {
-    const std::vector<uint64_t> ne(entries[i].shape.rbegin(), entries[i].shape.rend());  // innermost first
+    std::vector<uint64_t> ne(entries[i].shape.rbegin(), entries[i].shape.rend());  // innermost first
+    if (ne.empty()) ne.push_back(1);  // a single number
     rc = nfai_model_tensor_begin(m, need[i].name.c_str(), entries[i].dtype, ne.data(), (int)ne.size());
     if (rc == NFAI_OK) rc = nfai_model_tensor_chunk(m, entries[i].data, entries[i].bytes);
     if (rc == NFAI_OK) rc = nfai_model_tensor_end(m);

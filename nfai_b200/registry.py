@@ -20,7 +20,7 @@ def _open_planned(ctx: CudaContext, options: ModelOptions) -> CausalModel:
 
 
 # "architecture" of config.json -> how to open it
-CONFIG_ARCHITECTURES: Dict[str, Callable[[CudaContext, ModelOptions], CausalModel]] = {"Tometar": _open_planned}
+CONFIG_ARCHITECTURES: Dict[str, Callable[[CudaContext, ModelOptions], CausalModel]] = {"Tometar": _open_planned, "Tutizen": _open_planned}
 
 
 def architecture_of(path: str) -> str:
