@@ -162,7 +162,7 @@ int nfai_model_get_hparams(const nfai_model* m, nfai_hparams* out);
  * (post-norm residual, grouped-query attention with head norms, distance bias, head gates and borrowed keys and values,
  * clamped gated feed-forwards, dense or routed over experts). The handle is an
  * nfai_model like any other: prefill, decode, greedy and sampled loops, snapshots and taps work on it. Differences:
- * nfai_set_position only goes to 0 or the current position (recurrent state), one GPU, the cache has the weights' type,
+ * nfai_set_position goes back, with recurrent layers only to 0, one GPU, the cache has the weights' type,
  * nfai_read_kv returns the latent (kv_rank floats) as k and the shared rotated key part (rot_dim floats) as v of a latent
  * attention layer, and the normed heads (kv_heads * dim and kv_heads * vdim floats) of a grouped-query layer or the layer it
  * borrows from; nfai_read_hidden the sum of the streams. weight_dtype: NFAI_BF16 (served precision) or NFAI_F32 (true

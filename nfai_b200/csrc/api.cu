@@ -1235,8 +1235,8 @@ int nfai_set_position(nfai_model* m, uint32_t pos) {
   if (rc) return rc;
   if (pos > m->hp.ctx) return fail(m->ctx, NFAI_ERR_ARG, "position beyond the KV-cache capacity");
   // recurrent states cannot be rewound: only the start (states begin at zero there) and the current position
-  if (m->plan && pos != 0 && pos != m->pos)
-    return fail(m->ctx, NFAI_ERR_STATE, "a model with recurrent layers can only return to position 0; use a snapshot");
+  if (m->plan && pos != 0 && pos != m->pos && !(pos < m->pos && plan_rewinds(m)))
+    return fail(m->ctx, NFAI_ERR_STATE, "a model with recurrent layers can only return to position 0, others to an earlier one; use a snapshot");
   if ((rc = set_state_word(m, offsetof(StepState, pos), pos, 3))) return rc;
   CU(m->ctx, cudaStreamSynchronize(m->ctx->stream));
   m->pos = pos;

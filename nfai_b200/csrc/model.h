@@ -185,6 +185,7 @@ cudaError_t plan_record_step(nfai_model* m, bool with_head, bool from_prompt, in
 int plan_prefill(nfai_model* m, const uint32_t* tokens, int n, const uint32_t* want, int n_want, float* logits_out);
 bool plan_batched(const nfai_model* m);
 int plan_step_launches(const nfai_model* m);
+bool plan_rewinds(const nfai_model* m);  // every layer keeps rows per position: any earlier position can be returned to
 // settled: the residual behind the last layer is already in place (a prompt pass leaves it there)
 GemvParams plan_head_params(nfai_model* m, bool settled = false);
 size_t plan_snapshot_bytes(const nfai_model* m, uint32_t pos);

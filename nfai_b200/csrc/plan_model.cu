@@ -913,6 +913,12 @@ cudaError_t plan_record_step(nfai_model* m, bool with_head, bool from_prompt, in
 // (without graphs: known after the first recorded step)
 int plan_step_launches(const nfai_model* m) { return m->plan->step_launches; }
 
+bool plan_rewinds(const nfai_model* m) {
+  for (const PlanLayer& l : m->plan->plan.layers)
+    if (l.mixer == MIXER_SSM) return false;
+  return true;
+}
+
 // ---- prompt passes ----------------------------------------------------------------------------------------------------------------
 bool plan_batched(const nfai_model* m) { return m->plan->batched && m->plan->chunk >= 2; }
 

@@ -8,6 +8,7 @@
 #include <unistd.h>
 
 #include <string>
+#include <unordered_map>
 #include <vector>
 
 #include "../../include/nfai_cuda.h"
@@ -60,9 +61,11 @@ bool whole(const Json& j, uint64_t* out) {
   return true;
 }
 
-// The entry `name` of a parsed header; data sits behind `base`.
-bool find(const Json& header, const char* base, size_t avail, const std::string& name, Entry* e, std::string* err) {
-  const Json* t = header.get(name.c_str());
+// The entry `name` of a parsed header (indexed once: routed models have tens of thousands); data sits behind `base`.
+using Directory = std::unordered_map<std::string, const Json*>;
+bool find(const Directory& header, const char* base, size_t avail, const std::string& name, Entry* e, std::string* err) {
+  const auto it = header.find(name);
+  const Json* t = it == header.end() ? nullptr : it->second;
   if (!t) return *err = "model.safetensors has no tensor " + name, false;
   const Json *dt = t->get("dtype"), *sh = t->get("shape"), *of = t->get("data_offsets");
   const std::string bad = "model.safetensors: malformed entry of " + name;
@@ -104,13 +107,15 @@ extern "C" int nfai_model_load_dir(nfai_ctx* c, const char* dir, uint32_t kv_cac
   if (hlen > st.n - 8) return ctx_fail(c, NFAI_ERR_ARG, "model.safetensors is truncated");
   Json header;
   if (!JsonReader(st.p + 8, (size_t)hlen).parse(&header, &err)) return ctx_fail(c, NFAI_ERR_ARG, err.c_str());
+  Directory directory;
+  for (const auto& m : header.members) directory.emplace(m.first, &m.second);
   const char* base = st.p + 8 + hlen;
   const size_t avail = st.n - 8 - (size_t)hlen;
   // everything is looked up before a byte of device memory is taken
   const std::vector<PlanTensor> need = plan_tensors(plan);
   std::vector<Entry> entries(need.size());
   for (size_t i = 0; i < need.size(); ++i) {
-    if (!find(header, base, avail, need[i].name, &entries[i], &err)) return ctx_fail(c, NFAI_ERR_ARG, err.c_str());
+    if (!find(directory, base, avail, need[i].name, &entries[i], &err)) return ctx_fail(c, NFAI_ERR_ARG, err.c_str());
     if (entries[i].shape != need[i].shape) return ctx_fail(c, NFAI_ERR_ARG, ("tensor " + need[i].name + ": shape does not match config.json").c_str());
   }
   nfai_model* m = nullptr;
