@@ -18,9 +18,9 @@ Prints ONE JSON line on rank 0.
 
 --impl reference times that CPU port with all host threads on the same workload (rank 0 only).
 
---design tometar is a workload of its own (one GPU, one JSON line): prompt and decode throughput of Tometar models whose
-layers have a real model's sizes (random weights), each beside a Llama model of the same width, depth, feed-forward and
-vocabulary, with the decode kernels of both timed alone.
+--design tometar and --design tutizen are workloads of their own (one GPU, one JSON line): prompt and decode throughput of
+models of that design whose layers have a real model's sizes (random weights), each beside a Llama model of the same width,
+depth, feed-forward (per token) and vocabulary, with the decode kernels of both timed alone.
 """
 import argparse
 import json
@@ -437,7 +437,46 @@ def tometar_config(z):
     return {"architecture": "Tometar", "layers": layers, "norm": {"eps": 1e-5}, "streams": 4, "vocab": z["vocab"], "width": z["width"]}
 
 
-def tometar_tensors(cfg, seed):
+def tometar_params(z):
+    """Matrix elements of the layers that one token uses."""
+    la, sm, H, n = z["latent"], z["ssm"], z["width"], z["layers"]
+    p_la = (H * (la["heads"] * (la["dim"] + la["rot_dim"] + 2 * la["vdim"]) + la["kv_rank"] + la["rot_dim"])
+            + la["heads"] * (la["dim"] + la["vdim"]) * la["kv_rank"])
+    p_ss = H * (3 * sm["heads"] * sm["vdim"] + 2 * sm["groups"] * sm["state"] + sm["heads"])
+    return n // 2 * (p_la + p_ss) + n * 3 * H * z["ff"]
+
+
+# Dense layers with keys of their own and routed layers that borrow them, in turn; a token's share of a routed layer (chosen
+# and shared experts) is as wide as a dense feed-forward and as the Llama model's.
+TUTIZEN_SIZES = {
+    "1b": dict(width=2048, layers=16, ff=8192, vocab=128256, attn=dict(heads=32, kv_heads=8, dim=64, vdim=64),
+               moe=dict(experts=32, top=4, ff=1536, shared=2048, groups=4, keep=2), llama=dict(qH=32, kvH=8, d=64)),
+    "3b": dict(width=3072, layers=28, ff=8192, vocab=128256, attn=dict(heads=24, kv_heads=8, dim=128, vdim=128),
+               moe=dict(experts=64, top=6, ff=1024, shared=2048, groups=8, keep=4), llama=dict(qH=24, kvH=8, d=128)),
+}
+
+
+def tutizen_config(z):
+    at, mo = dict(z["attn"], scale=z["attn"]["dim"] ** -0.5), z["moe"]
+    routed = {"kind": "moe", "expert": {"ff": mo["ff"], "limit": 7.0}, "shared": {"ff": mo["shared"], "limit": 7.0},
+              "router": {"experts": mo["experts"], "top": mo["top"], "scale": 2.5, "groups": {"count": mo["groups"], "keep": mo["keep"]}}}
+    layers = [{"type": "attention", "mixer": at, "mlp": {"kind": "dense", "ff": z["ff"], "limit": 7.0}} if i % 2 == 0 else
+              {"type": "attention", "mixer": dict(at, kv_from=i - 1), "mlp": routed} for i in range(z["layers"])]
+    return {"architecture": "Tutizen", "layers": layers, "norm": {"eps": 1e-5}, "residual_mult": 0.5, "vocab": z["vocab"], "width": z["width"]}
+
+
+def tutizen_params(z):
+    at, mo, H, n = z["attn"], z["moe"], z["width"], z["layers"]
+    q, kv = H * (at["heads"] * (at["dim"] + at["vdim"] + 1)), H * at["kv_heads"] * (at["dim"] + at["vdim"])
+    routed = 3 * H * (mo["top"] * mo["ff"] + mo["shared"]) + H * (mo["experts"] + 1)
+    return n // 2 * (2 * q + kv + 3 * H * z["ff"] + routed)
+
+
+DESIGNS = {"tometar": ("Tometar", TOMETAR_SIZES, tometar_config, tometar_params),
+           "tutizen": ("Tutizen", TUTIZEN_SIZES, tutizen_config, tutizen_params)}
+
+
+def design_tensors(cfg, seed):
     """Random bfloat16 weights; large tensors repeat one block of normal draws from different places."""
     import numpy as np
 
@@ -458,6 +497,8 @@ def tometar_tensors(cfg, seed):
             v = np.linspace(0.0, 2.7, n, dtype=np.float32)
         elif last == "dt_bias":
             v = np.full(n, -4.0, np.float32)
+        elif last == "correction":
+            v = np.zeros(n, np.float32)
         elif last == "conv":
             v = block[:n] * 0.5
         else:
@@ -466,12 +507,13 @@ def tometar_tensors(cfg, seed):
         yield name, bits(v).reshape(shape), _lib.BF16
 
 
-def run_tometar(args):
+def run_design(args):
     import numpy as np
     import torch
 
     from nfai_b200 import LlamaModel, LlamaModelFactory, PlannedModel, synth, synthetic_tensors
     T, K = args.design_prompt, args.steps
+    title, all_sizes, config_of, params_of = DESIGNS[args.design]
     peak, peak_kind = measured_peak()
     sus, burst, _ = measured_tflops()
     factory = LlamaModelFactory(0)
@@ -512,40 +554,33 @@ def run_tometar(args):
         return {"prefill_tokens": T, "prefill_ms": pf * 1e3, "prefill_tok_s": T / pf, "decode_ms": step, "decode_tok_s": 1e3 / step,
                 "decode_e2e_tok_s": 1 / e2e, "launches_per_step": model.step_launches(), "kernels": kern}
 
+    def rates(r, params, z):
+        r["layer_matrix_params"] = params
+        r["weight_gb_per_step"] = 2 * (params + z["vocab"] * z["width"]) / 1e9
+        r["step_frac_of_copy_peak"] = r["weight_gb_per_step"] / (r["decode_ms"] * 1e-3) / peak
+        r["prefill_matrix_tflops"] = 2.0 * params * T / (r["prefill_ms"] * 1e-3) / 1e12
+        r["prefill_frac_of_sustained_bf16"] = r["prefill_matrix_tflops"] / sus
+        return r
+
     out = {}
     for size in args.sizes.split(","):
-        z = TOMETAR_SIZES[size]
-        cfg = tometar_config(z)
-        m = PlannedModel.from_tensors(factory.ctx, cfg, tometar_tensors(cfg, args.seed), T + K + 64, "bf16")
-        ours = measure(m, m.reset)
+        z = all_sizes[size]
+        cfg = config_of(z)
+        m = PlannedModel.from_tensors(factory.ctx, cfg, design_tensors(cfg, args.seed), T + K + 64, "bf16")
+        ours = rates(measure(m, m.reset), params_of(z), z)
         m.Dispose()
-        la, sm, H, n = z["latent"], z["ssm"], z["width"], z["layers"]
-        p_la = (H * (la["heads"] * (la["dim"] + la["rot_dim"] + 2 * la["vdim"]) + la["kv_rank"] + la["rot_dim"])
-                + la["heads"] * (la["dim"] + la["vdim"]) * la["kv_rank"])
-        inner = sm["heads"] * sm["vdim"]
-        p_ss = H * (3 * inner + 2 * sm["groups"] * sm["state"] + sm["heads"])
-        params = n // 2 * (p_la + p_ss) + n * 3 * H * z["ff"]
-        ours["layer_matrix_params"] = params
-        ours["weight_gb_per_step"] = 2 * (params + z["vocab"] * H) / 1e9
-        ours["step_frac_of_copy_peak"] = ours["weight_gb_per_step"] / (ours["decode_ms"] * 1e-3) / peak
-        ours["prefill_matrix_tflops"] = 2.0 * params * T / (ours["prefill_ms"] * 1e-3) / 1e12
-        ours["prefill_frac_of_sustained_bf16"] = ours["prefill_matrix_tflops"] / sus
-        lc = synth.ModelConfig(f"llama-{size}", H, n, z["llama"]["qH"], z["llama"]["kvH"], z["llama"]["d"], z["ff"], z["vocab"], "f16")
+        out[size] = {"config": z, args.design: ours}
+        if args.no_llama:
+            continue
+        lc = synth.ModelConfig(f"llama-{size}", z["width"], z["layers"], z["llama"]["qH"], z["llama"]["kvH"], z["llama"]["d"], z["ff"], z["vocab"], "f16")
         lm = LlamaModel(factory.ctx, synth.metadata(lc), synthetic_tensors(lc, args.seed), T + K + 64)
-        like = measure(lm, lm.reset)
+        out[size]["llama"] = rates(measure(lm, lm.reset), lc.streamed_matrix_params() - lc.V * lc.H, z)
         lm.Dispose()
-        lp = lc.streamed_matrix_params() - lc.V * lc.H
-        like["layer_matrix_params"] = lp
-        like["weight_gb_per_step"] = 2 * (lp + lc.V * lc.H) / 1e9
-        like["step_frac_of_copy_peak"] = like["weight_gb_per_step"] / (like["decode_ms"] * 1e-3) / peak
-        like["prefill_matrix_tflops"] = 2.0 * lp * T / (like["prefill_ms"] * 1e-3) / 1e12
-        like["prefill_frac_of_sustained_bf16"] = like["prefill_matrix_tflops"] / sus
-        out[size] = {"config": z, "tometar": ours, "llama": like}
     factory.Dispose()
-    print(json.dumps({"metric": "Tometar prompt and decode throughput (batch 1)", "unit": "tok/s", "n_gpus": 1, "steps": K, "data": "synthetic",
+    print(json.dumps({"metric": f"{title} prompt and decode throughput (batch 1)", "unit": "tok/s", "n_gpus": 1, "steps": K, "data": "synthetic",
                       "dtype": "bf16 weights and operands, f32 residual, norms, scores and state; Llama: f16", "peak_hbm_gbs": peak,
                       "peak_kind": peak_kind, "peak_bf16_tflops_sustained": sus, "sizes": out, "clocks": sampler.stop(),
-                      "l2": "every step streams all weights (larger than L2)"}), flush=True)
+                      "l2": "every step streams all weights it uses (larger than L2)"}), flush=True)
 
 
 def main():
@@ -564,12 +599,13 @@ def main():
     ap.add_argument("--nccl-allreduce", action="store_true", help="N > 1: use NCCL all-reduces instead of the peer-memory kernel")
     ap.add_argument("--prompt-len", type=int, default=0,
                     help="0 = the configuration's own prompt length (c1 128, c2 2048, c3 1024, c4 32768)")
-    ap.add_argument("--design", default="llama", choices=["llama", "tometar"], help="tometar: the workload described above")
-    ap.add_argument("--sizes", default="1b,3b", help="--design tometar: which of its sizes")
-    ap.add_argument("--design-prompt", type=int, default=2048, help="--design tometar: prompt length")
+    ap.add_argument("--design", default="llama", choices=["llama", *DESIGNS], help="the workloads described above")
+    ap.add_argument("--sizes", default="1b,3b", help="--design: which of its sizes")
+    ap.add_argument("--design-prompt", type=int, default=2048, help="--design: prompt length")
+    ap.add_argument("--no-llama", action="store_true", help="--design: leave out the Llama model beside it")
     args = ap.parse_args()
-    if args.design == "tometar":
-        run_tometar(args)
+    if args.design != "llama":
+        run_design(args)
         return
     global PROMPT_LEN, MIN_TIMED_S
     MIN_TIMED_S = args.min_timed_s

@@ -17,7 +17,7 @@ __host__ __device__ inline uint32_t gemv_x_floats(const GemvParams& p) {
   return (p.K * (1u + (p.gain ? 1u : 0u) + (p.post.y ? 1u : 0u)) + 3u) & ~3u;
 }
 __host__ __device__ inline uint32_t gemv_map_floats(const GemvParams& p, uint32_t vec_elems) {
-  if (p.map == MAP_EXPERT_ROWS) return 2 * kMaxChosen + kRouteScratch + p.expert.router.experts;
+  if (p.map == MAP_EXPERT_ROWS) return 2 * kMaxChosen + route_floats(p.expert.router.experts);
   if (p.map == MAP_EXPERT_COLUMNS) return 2 * (p.K / vec_elems);  // one pointer per vector of a row
   return 0;
 }
@@ -29,7 +29,7 @@ struct ChosenRows {  // MAP_EXPERT_ROWS
   __device__ __forceinline__ static void choose(const GemvParams& p, float* area) {
     if (threadIdx.x < 32) {
       uint32_t* const ids = reinterpret_cast<uint32_t*>(area);
-      route_warp(p.expert.router, p.expert.logits, area + 2 * kMaxChosen + kRouteScratch, area + 2 * kMaxChosen, ids, area + kMaxChosen);
+      route_warp(p.expert.router, p.expert.logits, area + 2 * kMaxChosen, ids, area + kMaxChosen);
       if (blockIdx.x == 0 && threadIdx.x < p.expert.router.top) p.expert.chosen[threadIdx.x] = ids[threadIdx.x];
     }
     __syncthreads();
@@ -39,18 +39,23 @@ struct ChosenRows {  // MAP_EXPERT_ROWS
     return (size_t)ids[k] * p.expert.rows + (n - k * p.expert.rows);
   }
 };
-// MAP_EXPERT_COLUMNS: element k of row 0; the rows of its matrix are *ld elements apart
+// MAP_EXPERT_COLUMNS: element k of row 0 of the matrix it belongs to; the rows of that matrix are *ld elements apart. `mine` is
+// the lane's entry of the chosen experts (chosen_lane). Every lane of the warp takes part.
+__device__ __forceinline__ uint32_t chosen_lane(const GemvParams& p) {
+  const uint32_t lane = threadIdx.x & 31;
+  return lane < p.expert.top ? __ldcg(p.expert.chosen + lane) : 0u;
+}
 template <typename WT>
-__device__ __forceinline__ const WT* chosen_column(const GemvParams& p, uint32_t k, uint32_t* ld) {
+__device__ __forceinline__ const WT* chosen_column(const GemvParams& p, uint32_t k, uint32_t mine, uint32_t* ld) {
   const ExpertMap& m = p.expert;
-  const uint32_t split = m.top * m.seg;
+  const uint32_t split = m.top * m.seg, i = min(k / m.seg, 31u);
+  const uint32_t e = __shfl_sync(0xffffffffu, mine, (int)i);
   if (k >= split) {
     *ld = p.K - split;
     return reinterpret_cast<const WT*>(m.W2) + (k - split);
   }
-  const uint32_t i = k / m.seg;
   *ld = m.seg;
-  return reinterpret_cast<const WT*>(p.W) + (size_t)__ldcg(m.chosen + i) * p.N * m.seg + (k - i * m.seg);
+  return reinterpret_cast<const WT*>(p.W) + (size_t)e * p.N * m.seg + (k - i * m.seg);
 }
 // x behind the experts' parts belongs to the shared feed-forward
 __device__ __forceinline__ void scale_shared(const GemvParams& p, float* xs) {
@@ -86,7 +91,8 @@ __global__ void __launch_bounds__(kThreads, 2) gemv_kernel(const GemvParams p) {
   const WT** const cols = reinterpret_cast<const WT**>(area);  // MAP_EXPERT_COLUMNS: vector v of row 0
   const uint32_t cols_split = MAP == MAP_EXPERT_COLUMNS ? p.expert.top * p.expert.seg / VE : 0u;
 
-  auto load_batch = [&](uint4(&buf)[U][R], uint32_t t, uint32_t kb) {
+  uint32_t mine = 0;  // MAP_EXPERT_COLUMNS, until the table of columns is there
+  auto load_batch = [&](uint4(&buf)[U][R], uint32_t t, uint32_t kb, bool first = false) {
     if (t >= nitems) return;
     const uint32_t rb = t >> sl, c = t & (S - 1);
     const uint32_t v0 = c * cv + kb * (32 * U) + lane;
@@ -95,7 +101,10 @@ __global__ void __launch_bounds__(kThreads, 2) gemv_kernel(const GemvParams p) {
 #pragma unroll
       for (int u = 0; u < U; ++u) {
         const uint32_t v = v0 + 32 * u;
-        const WT* col = v < vend ? cols[v] : nullptr;
+        uint32_t ld_first;
+        const WT* col = nullptr;
+        if (first) col = chosen_column<WT>(p, v * VE, mine, &ld_first);
+        else if (v < vend) col = cols[v];
         const uint32_t ld = v < cols_split ? p.expert.seg : p.K - p.expert.top * p.expert.seg;
 #pragma unroll
         for (int r = 0; r < R; ++r) {
@@ -139,17 +148,17 @@ __global__ void __launch_bounds__(kThreads, 2) gemv_kernel(const GemvParams p) {
   pdl_launch_dependents();
   pdl_wait();
   if constexpr (MAP != MAP_PLAIN) {  // which weights are needed is part of the previous kernel's result
-    if constexpr (MAP == MAP_EXPERT_ROWS) {
-      ChosenRows::choose(p, area);
-    } else {
-      for (uint32_t v = threadIdx.x; v < nvec; v += kThreads) {
-        uint32_t ld;
-        cols[v] = chosen_column<WT>(p, v * VE, &ld);
-      }
-      __syncthreads();
-    }
-    load_batch(cur, lt, lkb);
+    if constexpr (MAP == MAP_EXPERT_ROWS) ChosenRows::choose(p, area);
+    else mine = chosen_lane(p);
+    load_batch(cur, lt, lkb, true);
     advance();
+    if constexpr (MAP == MAP_EXPERT_COLUMNS) {  // read after the barriers of load_x
+      for (uint32_t v = threadIdx.x; v < ((nvec + 31u) & ~31u); v += kThreads) {
+        uint32_t ld;
+        const WT* col = chosen_column<WT>(p, v * VE, mine, &ld);
+        if (v < nvec) cols[v] = col;
+      }
+    }
   }
   // what the epilogue of the first item reads (residual / cos, sin of this position) travels with x
   uint32_t pos = 0;
@@ -256,6 +265,7 @@ __global__ void __launch_bounds__(kThreads) gemv_scalar_kernel(const GemvParams 
   float* const area = xs + gemv_x_floats(p);
   const ChosenRows rows(p, area);
   if constexpr (MAP == MAP_EXPERT_ROWS) ChosenRows::choose(p, area);
+  const uint32_t mine = MAP == MAP_EXPERT_COLUMNS ? chosen_lane(p) : 0u;
   load_x(p, xs, red);
   if constexpr (MAP == MAP_EXPERT_COLUMNS) scale_shared(p, xs);
   float best_v = -INFINITY;
@@ -267,10 +277,10 @@ __global__ void __launch_bounds__(kThreads) gemv_scalar_kernel(const GemvParams 
       uint32_t n = rb * R + r < p.N ? rb * R + r : p.N - 1;
       float a = 0.f;
       if constexpr (MAP == MAP_EXPERT_COLUMNS) {
-        for (uint32_t k = lane; k < p.K; k += 32) {
+        for (uint32_t k = lane; k < ((p.K + 31u) & ~31u); k += 32) {
           uint32_t ld;
-          const WT* col = chosen_column<WT>(p, k, &ld);
-          a = fmaf(to_float(col[(size_t)n * ld]), xs[k], a);
+          const WT* col = chosen_column<WT>(p, k, mine, &ld);
+          if (k < p.K) a = fmaf(to_float(col[(size_t)n * ld]), xs[k], a);
         }
       } else {
         const WT* w = reinterpret_cast<const WT*>(p.W) + (MAP == MAP_EXPERT_ROWS ? rows.row(p, n) : (size_t)n) * p.K;

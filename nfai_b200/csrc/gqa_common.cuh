@@ -27,7 +27,7 @@ __host__ __device__ __forceinline__ float slope2(const GqaSpec& s, uint32_t h) {
 // the rounding of cached rows) weighs less than 2^-64 of it: leaving those out is far below float32 rounding.
 __host__ __device__ __forceinline__ uint32_t reach(const GqaSpec& s, float slope_2) {
   if (!s.qk_norm || !s.distance_bias) return 0xffffffffu;
-  const float r = (2.04f * kLog2e * fabsf(s.scale) * (float)s.dim + 64.f) / slope_2;
+  const float r = (2.04f * kLog2e * fabsf(s.scale) * (float)s.dim + 40.f) / slope_2;
   return r < 4.0e9f ? (uint32_t)r + 1u : 0xffffffffu;
 }
 

@@ -7,6 +7,8 @@
 // A CTA of 16 warps owns up to GH query heads of one KV head and one range of positions; LPP lanes own one position (eight
 // elements each, NV times), so no shared memory and no barrier in the loop. Rows of earlier positions are requested before the
 // dependency wait. Splits are merged by the CTA that draws the last ticket of its heads; no CTA waits for another.
+#include <algorithm>
+
 #include "gqa_common.cuh"
 
 namespace nfai {
@@ -31,7 +33,7 @@ __global__ void __launch_bounds__(kGT, 1) gqa_decode_kernel(const GqaParams p, c
   using Raw = typename C8::Raw;
   constexpr int PPW = 32 / LPP;
   extern __shared__ __align__(16) float gsm[];  // [kGW][GH][vdim + 2]
-  __shared__ float fin_w[kGW][GH], fin_ML[GH][2], mw[GH][kSplitCap];
+  __shared__ float fin_w[kGW][GH], fin_ML[GH][2], mw[GH][kSplitCap], gates[GH];
   __shared__ uint32_t is_last;
   const GqaSpec& s = p.spec;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, grp = lane / LPP, sub = lane % LPP;
@@ -79,72 +81,94 @@ __global__ void __launch_bounds__(kGT, 1) gqa_decode_kernel(const GqaParams p, c
   pdl_wait();
   if (full && p.state && tid == 0) atomicOr(&p.state->err, 2u);
 
-  // eight elements (NV times) of a vector of `len` floats held by the lanes of a position; divided by the vector's root mean
-  // square when asked. Every lane of the warp takes part.
-  auto head_vector = [&](const float* src, uint32_t len, bool normed, float (&f)[NV][8]) {
-    float ss = 0.f;
+  // Eight elements (NV times) of a vector of `len` floats held by the lanes of a position, and the vector's division by its
+  // root mean square. Every lane of the warp takes part. All loads of the set-up are issued before the first sum.
+  auto fetch = [&](const float* src, uint32_t len, float (&f)[NV][8]) {
 #pragma unroll
     for (int v = 0; v < NV; ++v) {
       const int e0 = (v * LPP + sub) * 8;
+      if constexpr (VECT) {
+        const bool in = e0 < (int)len;
+        const float4 z = make_float4(0.f, 0.f, 0.f, 0.f);
+        const float4 a = in ? __ldcg(reinterpret_cast<const float4*>(src + e0)) : z, b = in ? __ldcg(reinterpret_cast<const float4*>(src + e0) + 1) : z;
+        f[v][0] = a.x; f[v][1] = a.y; f[v][2] = a.z; f[v][3] = a.w;
+        f[v][4] = b.x; f[v][5] = b.y; f[v][6] = b.z; f[v][7] = b.w;
+      } else {
 #pragma unroll
-      for (int e = 0; e < 8; ++e) {
-        f[v][e] = e0 + e < (int)len ? __ldcg(src + e0 + e) : 0.f;
-        ss = fmaf(f[v][e], f[v][e], ss);
+        for (int e = 0; e < 8; ++e) f[v][e] = e0 + e < (int)len ? __ldcg(src + e0 + e) : 0.f;
       }
     }
-    if (!normed) return;
-#pragma unroll
-    for (int o = 1; o < LPP; o <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-    const float rms = sqrtf(__fdiv_rn(ss, (float)len) + p.eps);
+  };
+  auto unit = [&](uint32_t len, float factor, float (&f)[NV][8]) {  // f / rms(f) * factor
+    float ss = 0.f;
 #pragma unroll
     for (int v = 0; v < NV; ++v)
 #pragma unroll
-      for (int e = 0; e < 8; ++e) f[v][e] = __fdiv_rn(f[v][e], rms);
+      for (int e = 0; e < 8; ++e) ss = fmaf(f[v][e], f[v][e], ss);
+#pragma unroll
+    for (int o = 1; o < LPP; o <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    const float c = __fdiv_rn(factor, sqrtf(__fdiv_rn(ss, (float)len) + p.eps));
+#pragma unroll
+    for (int v = 0; v < NV; ++v)
+#pragma unroll
+      for (int e = 0; e < 8; ++e) f[v][e] *= c;
   };
-  const bool own = s.own_kv();
+  const bool newest = t1 == pos + 1;  // this CTA's range ends with the new position
+  float q[GH][NV][8], sl[GH], m[GH], l[GH], acc[GH][NV][8], fk[NV][8], fv[NV][8];
   Raw new_k[NV], new_v[NV];
-  if (own) {
-    float f[NV][8];
-    head_vector(p.in + s.q_rows() + (size_t)g * dim, dim, s.qk_norm, f);
 #pragma unroll
-    for (int v = 0; v < NV; ++v) new_k[v] = C8::pack(f[v]);
-    head_vector(p.in + s.q_rows() + s.k_cols() + (size_t)g * vdim, vdim, s.v_norm, f);
-#pragma unroll
-    for (int v = 0; v < NV; ++v) new_v[v] = C8::pack(f[v]);
-    if (hg == 0 && t1 == pos + 1 && warp == 0 && grp == 0) {  // one CTA per KV head keeps the new rows
-      CT* ko = reinterpret_cast<CT*>(p.k_cache) + (size_t)pos * k_ld + (size_t)g * dim;
-      CT* vo = reinterpret_cast<CT*>(p.v_cache) + (size_t)pos * v_ld + (size_t)g * vdim;
+  for (int j = 0; j < GH; ++j) fetch(p.in + (size_t)(h0 + min((uint32_t)j, nh - 1)) * dim, dim, q[j]);  // (heads past the group repeat the last)
+  float gate_z = 0.f;
+  if (s.head_gate && (uint32_t)tid < nh) gate_z = __ldcg(p.in + s.gate_row0() + h0 + tid);
+  if (newest) {
+    if (s.own_kv()) {
+      fetch(p.in + s.q_rows() + (size_t)g * dim, dim, fk);
+      fetch(p.in + s.q_rows() + s.k_cols() + (size_t)g * vdim, vdim, fv);
+      if (s.qk_norm) unit(dim, 1.0f, fk);
+      if (s.v_norm) unit(vdim, 1.0f, fv);
 #pragma unroll
       for (int v = 0; v < NV; ++v) {
-        const int e0 = (v * LPP + sub) * 8;
-        C8::st(ko + e0, new_k[v], kn[v]);
-        C8::st(vo + e0, new_v[v], vn[v]);
+        new_k[v] = C8::pack(fk[v]);
+        new_v[v] = C8::pack(fv[v]);
       }
+      if (hg == 0 && warp == 0 && grp == 0) {  // one CTA per KV head keeps the new rows
+        CT* ko = reinterpret_cast<CT*>(p.k_cache) + (size_t)pos * k_ld + (size_t)g * dim;
+        CT* vo = reinterpret_cast<CT*>(p.v_cache) + (size_t)pos * v_ld + (size_t)g * vdim;
+#pragma unroll
+        for (int v = 0; v < NV; ++v) {
+          const int e0 = (v * LPP + sub) * 8;
+          C8::st(ko + e0, new_k[v], kn[v]);
+          C8::st(vo + e0, new_v[v], vn[v]);
+        }
+      }
+    } else {
+      load_rows(pos, true, new_k, new_v);  // the source layer of this step has written them
     }
-  } else {
-    load_rows(pos, true, new_k, new_v);  // the source layer of this step has written them
   }
-  float q[GH][NV][8], sl[GH], m[GH], l[GH], acc[GH][NV][8];
+  if (tid < GH) gates[tid] = s.head_gate ? head_sigmoid(gate_z) : 1.0f;  // (read behind the barriers of the merge)
 #pragma unroll
   for (int j = 0; j < GH; ++j) {
-    const uint32_t h = h0 + min((uint32_t)j, nh - 1);  // (heads past the group repeat the last one and are not stored)
-    head_vector(p.in + (size_t)h * dim, dim, s.qk_norm, q[j]);
-    sl[j] = slope2(s, h);
+    if (s.qk_norm) {
+      unit(dim, s.scale * kLog2e, q[j]);
+    } else {
+#pragma unroll
+      for (int v = 0; v < NV; ++v)
+#pragma unroll
+        for (int e = 0; e < 8; ++e) q[j][v][e] *= s.scale * kLog2e;
+    }
+    sl[j] = slope2(s, h0 + min((uint32_t)j, nh - 1));
     m[j] = kNegBig;
     l[j] = 0.f;
 #pragma unroll
     for (int v = 0; v < NV; ++v)
 #pragma unroll
-      for (int e = 0; e < 8; ++e) {
-        q[j][v][e] *= s.scale * kLog2e;
-        acc[j][v][e] = 0.f;
-      }
+      for (int e = 0; e < 8; ++e) acc[j][v][e] = 0.f;
   }
 
   while (base < t1) {
 #pragma unroll
     for (int u = 0; u < UNR; ++u)
-      if (base + u * (kGW * PPW) + grp == pos) {
+      if (newest && base + u * (kGW * PPW) + grp == pos) {
 #pragma unroll
         for (int v = 0; v < NV; ++v) {
           kr[u][v] = new_k[v];
@@ -234,25 +258,23 @@ __global__ void __launch_bounds__(kGT, 1) gqa_decode_kernel(const GqaParams p, c
     }
   }
   __syncthreads();
-  if (tid < GH) {
-    float M = kNegBig, L = 0.f;
-    for (int w = 0; w < kGW; ++w) M = fmaxf(M, gsm[(size_t)(w * GH + tid) * str + vdim]);
-    for (int w = 0; w < kGW; ++w) {
-      const float f = gqa_ex2(gsm[(size_t)(w * GH + tid) * str + vdim] - M);
-      fin_w[w][tid] = f;
-      L = fmaf(gsm[(size_t)(w * GH + tid) * str + vdim + 1], f, L);
+  if (warp < GH) {  // a warp per head, lanes along the warps' partials
+    const float* w = gsm + (size_t)((lane % kGW) * GH + warp) * str + vdim;
+    const float mw_l = lane < kGW ? w[0] : kNegBig, lw = lane < kGW ? w[1] : 0.f;
+    const float M = warp_max(mw_l), f = gqa_ex2(mw_l - M), L = warp_sum(lw * f);
+    if (lane < kGW) fin_w[lane][warp] = f;
+    if (lane == 0) {
+      fin_ML[warp][0] = M;
+      fin_ML[warp][1] = L;
     }
-    fin_ML[tid][0] = M;
-    fin_ML[tid][1] = L;
   }
   __syncthreads();
-  auto gate = [&](uint32_t j) { return s.head_gate ? head_sigmoid(__ldcg(p.in + s.gate_row0() + h0 + j)) : 1.0f; };
   for (uint32_t i = tid; i < nh * vdim; i += kGT) {
     const uint32_t j = i / vdim, e = i - j * vdim;
     float o = 0.f;
 #pragma unroll
     for (int w = 0; w < kGW; ++w) o = fmaf(gsm[(size_t)(w * GH + j) * str + e], fin_w[w][j], o);
-    if (S_eff == 1) p.out[(size_t)(h0 + j) * vdim + e] = o * __fdiv_rn(1.0f, fin_ML[j][1]) * gate(j);
+    if (S_eff == 1) p.out[(size_t)(h0 + j) * vdim + e] = o * __fdiv_rn(1.0f, fin_ML[j][1]) * gates[j];
     else d.part[((size_t)(h0 + j) * d.S_max + sp) * str + e] = o;
   }
   if (S_eff == 1) return;
@@ -261,21 +283,37 @@ __global__ void __launch_bounds__(kGT, 1) gqa_decode_kernel(const GqaParams p, c
     w[0] = fin_ML[tid][0];
     w[1] = fin_ML[tid][1];
   }
-  __threadfence();
   __syncthreads();
-  if (tid == 0) is_last = atomicAdd(&d.tickets[blockIdx.x], 1u) == S_eff - 1 ? 1u : 0u;
+  if (tid == 0) {
+    __threadfence();  // the block's stores, ordered before by the barrier, are out before the ticket ...
+    is_last = atomicAdd(&d.tickets[blockIdx.x], 1u) == S_eff - 1 ? 1u : 0u;
+    __threadfence();  // ... and the other blocks' are seen after it
+  }
   __syncthreads();
   if (!is_last) return;
-  __threadfence();
+  constexpr uint32_t kAhead = 8;  // partials a thread asks for before it uses one
+  float first[kAhead];            // those of its first output element, on their way while the weights are made
+  auto partial = [&](uint32_t i, uint32_t k) { return __ldcg(d.part + ((size_t)(h0 + i / vdim) * d.S_max + k) * str + i % vdim); };
+#pragma unroll
+  for (uint32_t k = 0; k < kAhead; ++k) first[k] = (uint32_t)tid < nh * vdim && k < S_eff ? partial(tid, k) : 0.f;
   for (uint32_t j = warp; j < nh; j += kGW) {
     const float* b = d.part + (size_t)(h0 + j) * d.S_max * str + vdim;
-    float M = kNegBig, L = 0.f;
-    for (uint32_t k = lane; k < S_eff; k += 32) M = fmaxf(M, __ldcg(b + (size_t)k * str));
+    constexpr int kPer = kSplitCap / 32;
+    float mk[kPer], lk[kPer], M = kNegBig, L = 0.f;
+#pragma unroll
+    for (int u = 0; u < kPer; ++u) {
+      const uint32_t k = lane + 32 * u;
+      mk[u] = k < S_eff ? __ldcg(b + (size_t)k * str) : kNegBig;
+      lk[u] = k < S_eff ? __ldcg(b + (size_t)k * str + 1) : 0.f;
+    }
+#pragma unroll
+    for (int u = 0; u < kPer; ++u) M = fmaxf(M, mk[u]);
     M = warp_max(M);
-    for (uint32_t k = lane; k < S_eff; k += 32) {
-      const float w = gqa_ex2(__ldcg(b + (size_t)k * str) - M);
-      mw[j][k] = w;
-      L = fmaf(__ldcg(b + (size_t)k * str + 1), w, L);
+#pragma unroll
+    for (int u = 0; u < kPer; ++u) {
+      const float w = gqa_ex2(mk[u] - M);
+      if (lane + 32 * u < S_eff) mw[j][lane + 32 * u] = w;
+      L = fmaf(lk[u], w, L);
     }
     L = warp_sum(L);
     if (lane == 0) fin_ML[j][1] = L;
@@ -283,11 +321,15 @@ __global__ void __launch_bounds__(kGT, 1) gqa_decode_kernel(const GqaParams p, c
   __syncthreads();
   for (uint32_t i = tid; i < nh * vdim; i += kGT) {
     const uint32_t j = i / vdim, e = i - j * vdim;
-    const float* b = d.part + (size_t)(h0 + j) * d.S_max * str + e;
     float o = 0.f;
+    uint32_t k = 0;
+    if (i == (uint32_t)tid) {
+#pragma unroll
+      for (; k < kAhead; ++k) o = fmaf(first[k], k < S_eff ? mw[j][k] : 0.f, o);
+    }
 #pragma unroll 8
-    for (uint32_t k = 0; k < S_eff; ++k) o = fmaf(__ldcg(b + (size_t)k * str), mw[j][k], o);
-    p.out[(size_t)(h0 + j) * vdim + e] = o * __fdiv_rn(1.0f, fin_ML[j][1]) * gate(j);
+    for (; k < S_eff; ++k) o = fmaf(partial(i, k), mw[j][k], o);
+    p.out[(size_t)(h0 + j) * vdim + e] = o * __fdiv_rn(1.0f, fin_ML[j][1]) * gates[j];
   }
   if (tid == 0) d.tickets[blockIdx.x] = 0;
 }
@@ -298,14 +340,22 @@ uint32_t heads_per_cta(const GqaSpec& s, uint32_t ctx) {
   if (ctx <= 4096 || G == 1 || s.dim > 128 || s.vdim > 128) return 1;
   return G <= 2 ? 2 : 4;
 }
+// As many splits of kMinChunk positions as a full cache needs, unless the CTAs with work would not fit the GPU at once; heads
+// whose bias keeps them near use fewer of them.
 DecodeShape decode_shape(const GqaSpec& s, uint32_t ctx, float* part) {
   DecodeShape d;
-  const uint32_t GH = heads_per_cta(s, ctx);
-  d.hgroups = (s.heads / s.kv_heads + GH - 1) / GH;
-  const uint32_t ctas = s.kv_heads * d.hgroups;
-  uint32_t S = (ctx + kMinChunk - 1) / kMinChunk;
-  if (S > sm_count() / ctas) S = sm_count() / ctas;
-  d.S_max = S < 1 ? 1 : S > kSplitCap ? kSplitCap : S;
+  const uint32_t GH = heads_per_cta(s, ctx), G = s.heads / s.kv_heads;
+  d.hgroups = (G + GH - 1) / GH;
+  uint32_t S = std::min((ctx + kMinChunk - 1) / kMinChunk, kSplitCap);
+  for (; S > 1; --S) {
+    const uint32_t chunk = std::max((ctx + S - 1) / S, kMinChunk);
+    uint64_t busy = 0;
+    for (uint32_t g = 0; g < s.kv_heads; ++g)
+      for (uint32_t i = 0; i < d.hgroups; ++i)
+        busy += (std::min<uint64_t>(ctx, (uint64_t)reach(s, slope2(s, g * G + std::min((i + 1) * GH, G) - 1)) + 1) + chunk - 1) / chunk;
+    if (busy <= sm_count()) break;
+  }
+  d.S_max = S < 1 ? 1 : S;
   d.part = part;
   d.tickets = reinterpret_cast<uint32_t*>(part + (size_t)s.heads * d.S_max * (s.vdim + 2));
   return d;

@@ -3,13 +3,19 @@
 //   gqa_prep           divides what the projection left by its root mean square, head by head: queries (times scale * log2 e)
 //                      become operands, keys and values cache rows. Lanes of a warp share a head in quads of elements.
 //   gqa_prefill_mma    flash attention on the warp-level tensor cores (bfloat16 operands, float32 accumulators) straight over
-//                      the cache: a CTA owns 16 tokens per warp of one head and walks the key tiles between the causal edge and
-//                      the reach of the head's distance bias (gqa_common.cuh). The bias is formed per key column relative to
-//                      the warp's first token: a constant per query changes nothing in its softmax, and the differences that
-//                      matter stay small numbers. Scores, exponentials and sums are float32, the weights enter the second
+//                      the cache: a CTA owns 64 tokens of one head and walks the key tiles from the causal edge back to the
+//                      reach of the head's distance bias (gqa_common.cuh). Two groups of four warps take alternate tiles and
+//                      are merged at the end: heads reach differently far, and the time of the launch is that of the longest
+//                      walk. Newest first: with a bias the running
+//                      maximum is then found early and the sums hardly ever have to be rescaled. A constant per query changes
+//                      nothing in its softmax, so the bias of a key is taken relative to the warp's first token: the part
+//                      inside a tile is what the score accumulators start from, the part of the tile itself goes into the
+//                      subtraction of the maximum. Scores, exponentials and sums are float32, the weights enter the second
 //                      product as a bfloat16 head and remainder (relative error ~2^-17).
 //   gqa_prefill_simt   the same for true float32 and for head sizes the former does not take.
 // A portion may start anywhere: earlier positions are read from the cache.
+#include <algorithm>
+
 #include "gqa_common.cuh"
 
 namespace nfai {
@@ -125,8 +131,9 @@ __device__ __forceinline__ void cpa16(uint32_t dst, const void* src, uint32_t by
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(bytes) : "memory");
 }
 
-constexpr int kPW = 8, kPM = kPW * 16, kPThr = kPW * 32;  // warps and tokens per CTA
-constexpr int kPBuf = 3;                                  // tile buffers: two in flight while one is multiplied
+constexpr int kPGroups = 2, kPW = 4;                              // groups of warps, warps of a group
+constexpr int kPM = kPW * 16, kPThr = kPGroups * kPW * 32;        // tokens and threads of a CTA
+constexpr int kPBuf = 2 * kPGroups;                               // tile buffers: a tile per group, and the next ones in flight
 
 // DQ > 0: dim padded to it, query fragments stay in registers; DQ = 0: any dim, the query is read from shared memory per tile.
 template <int DQ, int DV, int kN>
@@ -143,8 +150,8 @@ __global__ void __launch_bounds__(kPThr, DV <= 64 && DQ == 64 ? 2 : 1) gqa_prefi
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, qr = lane >> 2, qc = (lane & 3) * 2;
   pdl_launch_dependents();
   pdl_wait();
-  // the last tiles of tokens (the longest) of all heads start first
-  const uint32_t h = blockIdx.x % s.heads, tile = gridDim.x / s.heads - 1 - blockIdx.x / s.heads, g = h / (s.heads / s.kv_heads);
+  // the last tiles of tokens of the heads that reach farthest start first
+  const uint32_t h = s.heads - 1 - blockIdx.x % s.heads, tile = gridDim.x / s.heads - 1 - blockIdx.x / s.heads, g = h / (s.heads / s.kv_heads);
   const uint32_t t0 = tile * kPM, rows_end = min(T, t0 + kPM);
   const uint32_t first_pos = p.pos0 + t0, k_hi = p.pos0 + rows_end;  // one past the last visible position
   const float sl = slope2(s, h);
@@ -180,42 +187,50 @@ __global__ void __launch_bounds__(kPThr, DV <= 64 && DQ == 64 ? 2 : 1) gqa_prefi
   };
   stage(Qs, LQ, Q, q_ld, t0, kPM, T, dim, DQr);
   const uint32_t ntiles = (k_hi - k_lo + kN - 1) / kN;
-  issue(0, k_lo);
-  asm volatile("cp.async.commit_group;" ::: "memory");  // the query rows and the first tile
-  if (ntiles > 1) issue(1, k_lo + kN);
-  asm volatile("cp.async.commit_group;" ::: "memory");
+  auto tile_pos = [&](uint32_t it) { return k_lo + (ntiles - 1 - it) * kN; };  // newest first
+  auto issue_round = [&](uint32_t round) {  // a tile for each group
+#pragma unroll
+    for (int i = 0; i < kPGroups; ++i)
+      if (round * kPGroups + i < ntiles) issue((round & 1u) * kPGroups + i, tile_pos(round * kPGroups + i));
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  issue_round(0);  // with the query rows
 
-  const uint32_t row_a = t0 + warp * 16 + qr, row_b = row_a + 8;
+  const int group = warp / kPW, wq = warp % kPW;  // this warp's group, and its place among the tokens
+  const uint32_t row_a = t0 + wq * 16 + qr, row_b = row_a + 8;
   const uint32_t pos_a = p.pos0 + row_a, pos_b = p.pos0 + row_b;
-  const uint32_t w_first = first_pos + warp * 16, w_last = w_first + 15;
+  const uint32_t w_first = first_pos + wq * 16, w_last = w_first + 15;
   float o[DV / 8][4];
 #pragma unroll
   for (int j = 0; j < DV / 8; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
   float m_a = kNegBig, m_b = kNegBig, l_a = 0.f, l_b = 0.f;
   const int lm = lane >> 3, lr = lane & 7;
-  const uint32_t q_s = (uint32_t)__cvta_generic_to_shared(Qs) + (uint32_t)((warp * 16 + (lm & 1) * 8 + lr) * LQ + (lm >> 1) * 8) * 2;
+  const uint32_t q_s = (uint32_t)__cvta_generic_to_shared(Qs) + (uint32_t)((wq * 16 + (lm & 1) * 8 + lr) * LQ + (lm >> 1) * 8) * 2;
   const uint32_t k_off = (uint32_t)(((lm >> 1) * 8 + lr) * LQ + (lm & 1) * 8) * 2;
   const uint32_t v_off = (uint32_t)(((lm & 1) * 8 + lr) * LV + (lm >> 1) * 8) * 2;
   const uint32_t ks_b = (uint32_t)__cvta_generic_to_shared(Ks), vs_b = (uint32_t)__cvta_generic_to_shared(Vs);
   uint32_t qf[DQ ? DQ / 16 : 1][4];
+  const float b_lane = sl * (float)qc;
 
-  for (uint32_t it = 0; it < ntiles; ++it) {
-    const uint32_t kb = k_lo + it * kN, buf = it % kPBuf;
-    asm volatile("cp.async.wait_group 1;" ::: "memory");
-    __syncthreads();  // tile `it` is there for every warp, and every warp has left tile it - 1
-    if (it + 2 < ntiles) issue((it + 2) % kPBuf, kb + 2 * kN);
-    asm volatile("cp.async.commit_group;" ::: "memory");
+  for (uint32_t round = 0; round * kPGroups < ntiles; ++round) {
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();  // this round's tiles are there for every warp, and every warp has left the last round's
+    if ((round + 1) * kPGroups < ntiles) issue_round(round + 1);
+    const uint32_t it = round * kPGroups + group, buf = (round & 1u) * kPGroups + group, kb = tile_pos(it < ntiles ? it : 0);
     if constexpr (DQ > 0) {
-      if (it == 0) {
+      if (round == 0) {
 #pragma unroll
         for (int kk = 0; kk < DQ / 16; ++kk) ldsm4(q_s + kk * 32, qf[kk]);
       }
     }
-    if (kb > w_last) continue;  // (warp-uniform)
+    if (it >= ntiles || kb > w_last) continue;  // (warp-uniform)
     const uint32_t ks = ks_b + buf * (uint32_t)(kN * LQ * 2), vs = vs_b + buf * (uint32_t)(kN * LV * 2);
     float c[kN / 8][4];
 #pragma unroll
-    for (int j = 0; j < kN / 8; ++j) c[j][0] = c[j][1] = c[j][2] = c[j][3] = 0.f;
+    for (int j = 0; j < kN / 8; ++j) {  // (without a bias sl is zero)
+      c[j][0] = c[j][2] = fmaf(sl, (float)(j * 8), b_lane);
+      c[j][1] = c[j][3] = fmaf(sl, (float)(j * 8 + 1), b_lane);
+    }
     auto scores = [&](const uint32_t (&a)[4], uint32_t kk) {
 #pragma unroll
       for (int j = 0; j < kN / 8; j += 2) {
@@ -233,17 +248,6 @@ __global__ void __launch_bounds__(kPThr, DV <= 64 && DQ == 64 ? 2 : 1) gqa_prefi
         uint32_t a[4];
         ldsm4(q_s + kk * 32, a);
         scores(a, kk);
-      }
-    }
-    if (s.distance_bias) {
-      const float rel = (float)((int)(kb + qc) - (int)w_first);  // position of this lane's first column, from the warp's first token
-#pragma unroll
-      for (int j = 0; j < kN / 8; ++j) {
-        const float b0 = sl * (rel + (float)(j * 8)), b1 = sl * (rel + (float)(j * 8 + 1));
-        c[j][0] += b0;
-        c[j][1] += b1;
-        c[j][2] += b0;
-        c[j][3] += b1;
       }
     }
     if (kb + kN - 1 > w_first) {  // not every row of the warp sees the whole tile
@@ -266,10 +270,23 @@ __global__ void __launch_bounds__(kPThr, DV <= 64 && DQ == 64 ? 2 : 1) gqa_prefi
     mx_a = fmaxf(mx_a, __shfl_xor_sync(0xffffffffu, mx_a, 2));
     mx_b = fmaxf(mx_b, __shfl_xor_sync(0xffffffffu, mx_b, 1));
     mx_b = fmaxf(mx_b, __shfl_xor_sync(0xffffffffu, mx_b, 2));
-    const float mn_a = fmaxf(m_a, mx_a), mn_b = fmaxf(m_b, mx_b);
-    const float al_a = gqa_ex2(m_a - mn_a), al_b = gqa_ex2(m_b - mn_b);
-    m_a = mn_a;
-    m_b = mn_b;
+    const float tile_bias = sl * (float)((int)kb - (int)w_first);
+    const float new_a = fmaxf(m_a, mx_a + tile_bias), new_b = fmaxf(m_b, mx_b + tile_bias);
+    if (__any_sync(0xffffffffu, new_a > m_a || new_b > m_b)) {
+      const float al_a = gqa_ex2(m_a - new_a), al_b = gqa_ex2(m_b - new_b);
+      m_a = new_a;
+      m_b = new_b;
+      l_a *= al_a;
+      l_b *= al_b;
+#pragma unroll
+      for (int j = 0; j < DV / 8; ++j) {
+        o[j][0] *= al_a;
+        o[j][1] *= al_a;
+        o[j][2] *= al_b;
+        o[j][3] *= al_b;
+      }
+    }
+    const float mn_a = m_a - tile_bias, mn_b = m_b - tile_bias;
     float sum_a = 0.f, sum_b = 0.f;
     uint32_t ph[kN / 16][4], pl[kN / 16][4];
 #pragma unroll
@@ -284,15 +301,8 @@ __global__ void __launch_bounds__(kPThr, DV <= 64 && DQ == 64 ? 2 : 1) gqa_prefi
       pl[i][w] = pack_bf(e0 - __uint_as_float(ha << 16), e1 - __uint_as_float(ha & 0xffff0000u));
       pl[i][w + 1] = pack_bf(e2 - __uint_as_float(hb << 16), e3 - __uint_as_float(hb & 0xffff0000u));
     }
-    l_a = l_a * al_a + sum_a;
-    l_b = l_b * al_b + sum_b;
-#pragma unroll
-    for (int j = 0; j < DV / 8; ++j) {
-      o[j][0] *= al_a;
-      o[j][1] *= al_a;
-      o[j][2] *= al_b;
-      o[j][3] *= al_b;
-    }
+    l_a += sum_a;
+    l_b += sum_b;
 #pragma unroll
     for (int kk = 0; kk < kN / 16; ++kk) {
 #pragma unroll
@@ -306,7 +316,33 @@ __global__ void __launch_bounds__(kPThr, DV <= 64 && DQ == 64 ? 2 : 1) gqa_prefi
       }
     }
   }
-  asm volatile("cp.async.wait_group 0;" ::: "memory");
+  // the second group's sums join the first's (the buffers are free: nothing is in flight any more)
+  static_assert(kPGroups == 2, "one group hands over to the other");
+  __syncthreads();
+  float* const hand = reinterpret_cast<float*>(Ks);  // [DV/8 + 1][kPW * 32] quads
+  const int slot = (wq * 32 + lane) * 4;
+  if (group == 1) {
+#pragma unroll
+    for (int j = 0; j < DV / 8; ++j) *reinterpret_cast<float4*>(hand + j * (kPW * 128) + slot) = make_float4(o[j][0], o[j][1], o[j][2], o[j][3]);
+    *reinterpret_cast<float4*>(hand + DV / 8 * (kPW * 128) + slot) = make_float4(m_a, m_b, l_a, l_b);
+  }
+  __syncthreads();
+  if (group == 1) return;
+  {
+    const float4 r = *reinterpret_cast<const float4*>(hand + DV / 8 * (kPW * 128) + slot);
+    const float M_a = fmaxf(m_a, r.x), M_b = fmaxf(m_b, r.y);
+    const float x_a = gqa_ex2(m_a - M_a), x_b = gqa_ex2(m_b - M_b), y_a = gqa_ex2(r.x - M_a), y_b = gqa_ex2(r.y - M_b);
+    l_a = l_a * x_a + r.z * y_a;
+    l_b = l_b * x_b + r.w * y_b;
+#pragma unroll
+    for (int j = 0; j < DV / 8; ++j) {
+      const float4 v = *reinterpret_cast<const float4*>(hand + j * (kPW * 128) + slot);
+      o[j][0] = o[j][0] * x_a + v.x * y_a;
+      o[j][1] = o[j][1] * x_a + v.y * y_a;
+      o[j][2] = o[j][2] * x_b + v.z * y_b;
+      o[j][3] = o[j][3] * x_b + v.w * y_b;
+    }
+  }
   l_a += __shfl_xor_sync(0xffffffffu, l_a, 1);
   l_a += __shfl_xor_sync(0xffffffffu, l_a, 2);
   l_b += __shfl_xor_sync(0xffffffffu, l_b, 1);
@@ -331,7 +367,10 @@ __global__ void __launch_bounds__(kPThr, DV <= 64 && DQ == 64 ? 2 : 1) gqa_prefi
   }
 }
 
-size_t prefill_smem(uint32_t DQ, uint32_t DV, uint32_t kN) { return ((size_t)(kPM + kPBuf * kN) * (DQ + 8) + (size_t)kPBuf * kN * (DV + 8)) * 2; }
+size_t prefill_smem(uint32_t DQ, uint32_t DV, uint32_t kN) {
+  const size_t q = (size_t)kPM * (DQ + 8) * 2, tiles = (size_t)kPBuf * kN * (DQ + DV + 16) * 2, hand = (size_t)(DV / 8 + 1) * kPW * 128 * 4;
+  return q + std::max(tiles, hand);
+}
 uint32_t value_width(uint32_t vdim) { return vdim <= 32 ? 32 : vdim <= 64 ? 64 : vdim <= 128 ? 128 : vdim <= 256 ? 256 : 0; }
 
 template <int DQ, int DV, int kN>

@@ -17,13 +17,12 @@ constexpr int kCW = 8;    // warps (tokens) per CTA of moe_choose
 constexpr int kST = 512;  // threads of moe_sort
 
 __global__ void __launch_bounds__(kCW * 32) moe_choose_kernel(const MoeRows p, const uint32_t T) {
-  extern __shared__ float csm[];  // per warp: [experts] scores, kRouteScratch
+  extern __shared__ float csm[];  // route_floats(experts) per warp
   pdl_launch_dependents();
   pdl_wait();
-  const uint32_t warp = threadIdx.x >> 5, t = blockIdx.x * kCW + warp, per = p.router.experts + kRouteScratch;
+  const uint32_t warp = threadIdx.x >> 5, t = blockIdx.x * kCW + warp;
   if (t >= T) return;
-  float* cs = csm + warp * per;
-  route_warp(p.router, p.logits + (size_t)t * p.ld, cs, cs + p.router.experts, p.ids + (size_t)t * p.router.top, p.w + (size_t)t * p.router.top);
+  route_warp(p.router, p.logits + (size_t)t * p.ld, csm + warp * route_floats(p.router.experts), p.ids + (size_t)t * p.router.top, p.w + (size_t)t * p.router.top);
 }
 
 // exclusive prefix sum over the CTA; *total receives the sum
@@ -76,17 +75,27 @@ __global__ void __launch_bounds__(kST) moe_sort_kernel(const MoeRows p, const ui
     }
   }
   for (uint32_t i = tid; i < my_tiles; i += kST) p.tiles[tile0 + i] = make_uint2(e, row0 + i * kGroupTile);
-  // this expert's pairs, in order
-  uint32_t at = row0;
-  for (uint32_t base = 0; base < n; base += kST) {
-    const uint32_t i = base + tid;
-    const bool hit = i < n && min(p.ids[i], E - 1) == e;
-    const uint32_t rank = cta_prefix(hit ? 1u : 0u, sums, &any);
+  // this expert's pairs, in order: a warp takes a run of them, counts its hits, and ranks them behind the earlier warps'
+  const uint32_t lane = tid & 31, warp = tid >> 5, run = ((n + kST / 32 - 1) / (kST / 32) + 31) & ~31u;
+  const uint32_t i0 = min(warp * run, n), i1 = min(i0 + run, n);
+  uint32_t hits = 0;
+#pragma unroll 4
+  for (uint32_t i = i0 + lane; i < i1; i += 32) hits += min(p.ids[i], E - 1) == e ? 1u : 0u;
+  hits = __reduce_add_sync(0xffffffffu, hits);
+  uint32_t at = row0 + cta_prefix(lane == 0 ? hits : 0u, sums, &any);
+  at = __shfl_sync(0xffffffffu, at, 0);
+  if (!hits) return;
+#pragma unroll 4
+  for (uint32_t base = i0; base < i1; base += 32) {
+    const uint32_t i = base + lane;
+    const bool hit = i < i1 && min(p.ids[i], E - 1) == e;
+    const uint32_t mask = __ballot_sync(0xffffffffu, hit);
     if (hit) {
-      p.where[i] = at + rank;
-      p.src[at + rank] = i / top;
+      const uint32_t to = at + __popc(mask & ((1u << lane) - 1u));
+      p.where[i] = to;
+      p.src[to] = i / top;
     }
-    at += any;
+    at += __popc(mask);
   }
 }
 
@@ -107,7 +116,7 @@ cudaError_t launch_moe_route(cudaStream_t s, const MoeRows& p, uint32_t T) {
   const Router& r = p.router;
   if (!T || !r.experts || r.experts > kMaxExperts || !r.top || r.top > kMaxChosen || r.groups > kMaxGroups || !r.groups || r.experts % r.groups)
     return cudaErrorInvalidValue;
-  const size_t smem = (size_t)kCW * (r.experts + kRouteScratch) * 4;
+  const size_t smem = (size_t)kCW * route_floats(r.experts) * 4;
   cudaError_t e = cudaSuccess;
   if (smem > 40 * 1024 &&
       (e = cudaFuncSetAttribute(moe_choose_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)) != cudaSuccess)

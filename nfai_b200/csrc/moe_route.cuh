@@ -20,14 +20,21 @@ __device__ __forceinline__ uint32_t ordered_bits(float v) {
 }
 __device__ __forceinline__ float route_sigmoid(float z) { return __fdiv_rn(1.0f, 1.0f + expf(-z)); }
 
-constexpr uint32_t kRouteScratch = kMaxGroups;  // floats beside the experts' scores
+constexpr uint32_t kRouteScratch = kMaxGroups;  // floats beside the experts' scores and choice scores
+constexpr uint32_t route_floats(uint32_t experts) { return 2 * experts + kRouteScratch; }
 
-// cs: [experts] and gs: [kRouteScratch] floats of shared memory of this warp; ids and w: [top], shared memory or global.
-// Every lane calls it; the results are visible to the warp when it returns.
-__device__ __forceinline__ void route_warp(const Router& r, const float* z, float* cs, float* gs, uint32_t* ids, float* w) {
+// scratch: route_floats(experts) floats of shared memory of this warp; ids and w: [top], shared memory or global. Every lane
+// calls it; the results are visible to the warp when it returns.
+__device__ __forceinline__ void route_warp(const Router& r, const float* z, float* scratch, uint32_t* ids, float* w) {
   const uint32_t lane = threadIdx.x & 31, E = r.experts;
   constexpr uint32_t kAll = 0xffffffffu;
-  for (uint32_t e = lane; e < E; e += 32) cs[e] = route_sigmoid(__ldcg(z + e)) + __ldg(r.correction + e);
+  float *const gs = scratch, *const cs = gs + kRouteScratch, *const sc = cs + E;
+#pragma unroll 4
+  for (uint32_t e = lane; e < E; e += 32) {
+    const float s = route_sigmoid(__ldcg(z + e));
+    sc[e] = s;
+    cs[e] = s + __ldg(r.correction + e);
+  }
   __syncwarp();
   if (r.keep < r.groups) {
     const uint32_t size = E / r.groups;
@@ -85,7 +92,7 @@ __device__ __forceinline__ void route_warp(const Router& r, const float* z, floa
       cs[e] = -INFINITY;
       scan();
     }
-    const float s = route_sigmoid(__ldcg(z + e));
+    const float s = sc[e];
     sum += s;
     if (lane == k) {
       mine = s;
