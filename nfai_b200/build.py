@@ -21,7 +21,7 @@ LIB_DIR = os.path.join(HERE, "lib")
 LIB_PATH = os.path.join(LIB_DIR, "libnfai_cuda.so")
 INCLUDE = os.path.join(os.path.dirname(HERE), "include")
 
-SOURCES = ["api.cu", "gemv.cu", "gemv_bf16.cu", "gemv_moe.cu", "gemv_ring.cu", "gemm_tc.cu", "gemm_simt.cu", "attn.cu", "attn_ring.cu", "attn_mma.cu", "attn_prefill_tc.cu", "attn_static.cu", "misc.cu", "tp.cu", "gguf_loader.cu", "sample.cu", "tokenizer.cpp",
+SOURCES = ["api.cu", "gemv.cu", "gemv_bf16.cu", "gemv_post.cu", "gemv_moe.cu", "gemv_ring.cu", "gemm_tc.cu", "gemm_simt.cu", "attn.cu", "attn_ring.cu", "attn_mma.cu", "attn_prefill_tc.cu", "attn_static.cu", "misc.cu", "tp.cu", "gguf_loader.cu", "sample.cu", "tokenizer.cpp",
            "plan.cpp", "plan_model.cu", "safetensors_loader.cpp", "hyper.cu", "latent.cu", "latent_decode_mma.cu", "latent_prefill.cu", "ssm.cu", "ssm_chunk.cu", "post_rows.cu", "gqa_decode.cu", "gqa_prefill.cu", "moe.cu"]
 
 NVCC_FLAGS = [

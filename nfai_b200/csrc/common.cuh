@@ -136,15 +136,16 @@ __device__ __forceinline__ void store_as(float* p, float v) { *p = v; }
 __device__ __forceinline__ void store_as(__half* p, float v) { *p = __float2half_rn(v); }
 __device__ __forceinline__ void store_as(__nv_bfloat16* p, float v) { *p = __float2bfloat16_rn(v); }
 
-// Gated feed-forward: up * act(gate), act = silu or relu (Activation in kernels.h), or the clamped form
-// g sigmoid(1.702 g) (u + 1) with g = min(gate, limit) and u = up held to +-limit. silu keeps the operation order
+// The clamped gated activation g sigmoid(1.702 g) (u + 1) with g = min(gate, limit) and u = up held to +-limit.
+__device__ __forceinline__ float gated_clamped(float gate, float up, float limit) {
+  const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
+  return g * __fdiv_rn(1.0f, 1.0f + expf(-1.702f * g)) * (u + 1.0f);
+}
+
+// Gated feed-forward: up * act(gate), act = silu or relu (Activation in kernels.h). silu keeps the operation order
 // sigmoid = 1/(1+exp(-x)), x*sigmoid, up*silu.
-__device__ __forceinline__ float gated(int act, float gate, float up, float limit) {
+__device__ __forceinline__ float gated(int act, float gate, float up) {
   if (act == 1) return __fmul_rn(up, fmaxf(gate, 0.f));
-  if (act == 2) {
-    const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
-    return g * __fdiv_rn(1.0f, 1.0f + expf(-1.702f * g)) * (u + 1.0f);
-  }
   const float sig = __fdiv_rn(1.0f, 1.0f + expf(-gate));
   return __fmul_rn(up, __fmul_rn(gate, sig));
 }

@@ -66,12 +66,13 @@ __device__ __forceinline__ void epilogue_pair(const GemmEpilogue& ep, uint32_t m
       break;
     }
     case GEMM_EPI_GATED: {  // columns (2j, 2j+1) = (gate_j, up_j); h_j = up * act(gate)
-      if (ep.gated_cols && n >= ep.gated_cols) {  // plain columns behind the gated ones (both counts are even)
-        *reinterpret_cast<float2*>(ep.out_f32 + (size_t)m * (N - ep.gated_cols) + (n - ep.gated_cols)) = make_float2(a, b);
-        break;
-      }
-      if (n + 1 < N)
-        store_operand(ep, (size_t)m * ((ep.gated_cols ? ep.gated_cols : N) / 2) + (n >> 1), gated(ep.act, a + aux.x, b + aux.y, ep.act_limit));
+      if (n + 1 < N) store_operand(ep, (size_t)m * (N / 2) + (n >> 1), gated(ep.act, a + aux.x, b + aux.y));
+      break;
+    }
+    case GEMM_EPI_GATED_CLAMPED: {
+      const uint32_t cols = ep.gated_cols ? ep.gated_cols : N;
+      if (n < cols) store_operand(ep, (size_t)m * (cols / 2) + (n >> 1), gated_clamped(a, b, ep.act_limit));
+      else *reinterpret_cast<float2*>(ep.out_f32 + (size_t)m * (N - cols) + (n - cols)) = make_float2(a, b);
       break;
     }
     case GEMM_EPI_STORE_ACT: {  // plain store in the operand type of the next product

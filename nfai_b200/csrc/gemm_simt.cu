@@ -79,7 +79,7 @@ __global__ void __launch_bounds__(256) gemm_simt_kernel(const T* __restrict__ A,
 
 cudaError_t launch_gemm_simt(cudaStream_t s, int dtype, const void* A, const void* W, uint32_t M, uint32_t N, uint32_t K,
                              const GemmEpilogue& ep) {
-  if (!A || !W || !M || !N || !K || (ep.kind == GEMM_EPI_GATED && (N & 1u))) return cudaErrorInvalidValue;
+  if (!A || !W || !M || !N || !K || ((ep.kind == GEMM_EPI_GATED || ep.kind == GEMM_EPI_GATED_CLAMPED) && (N & 1u))) return cudaErrorInvalidValue;
   const dim3 grid((N + kT - 1) / kT, (M + kT - 1) / kT);
   const GemmGroups none;
   if (dtype == 0)
@@ -92,7 +92,7 @@ cudaError_t launch_gemm_simt(cudaStream_t s, int dtype, const void* A, const voi
 
 cudaError_t launch_gemm_simt_grouped(cudaStream_t s, int dtype, const void* A, const void* W, uint32_t N, uint32_t K, const GemmGroups& g,
                                      const GemmEpilogue& ep) {
-  if (!A || !W || !N || !K || !g.max_tiles || ep.bias || ep.resid || (ep.kind == GEMM_EPI_GATED && (N & 1u))) return cudaErrorInvalidValue;
+  if (!A || !W || !N || !K || !g.max_tiles || ep.bias || ep.resid || ((ep.kind == GEMM_EPI_GATED || ep.kind == GEMM_EPI_GATED_CLAMPED) && (N & 1u))) return cudaErrorInvalidValue;
   const dim3 grid((N + kT - 1) / kT, g.max_tiles * (kGroupTile / kT));
   if (grid.y > 65535) return cudaErrorInvalidValue;
   if (dtype == 0)

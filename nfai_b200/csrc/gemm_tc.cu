@@ -528,6 +528,7 @@ __global__ void __launch_bounds__(kPThreadsGemm) gemm_tc_persistent_kernel(const
       };
       switch (ep.kind) {
         case GEMM_EPI_STORE: ok = tile_epilogue(std::integral_constant<int, (int)GEMM_EPI_STORE>{}); break;
+        case GEMM_EPI_GATED_CLAMPED: ok = tile_epilogue(std::integral_constant<int, (int)GEMM_EPI_GATED_CLAMPED>{}); break;
         case GEMM_EPI_GATED: ok = tile_epilogue(std::integral_constant<int, (int)GEMM_EPI_GATED>{}); break;
         case GEMM_EPI_STORE_ACT: ok = tile_epilogue(std::integral_constant<int, (int)GEMM_EPI_STORE_ACT>{}); break;
         default: ok = tile_epilogue(std::integral_constant<int, (int)GEMM_EPI_QKV_ROPE>{}); break;
@@ -699,7 +700,7 @@ uint32_t gemm_tc_splits(uint32_t M, uint32_t N, uint32_t K) {
 cudaError_t launch_gemm_tc(cudaStream_t s, const __half* A, const __half* W, uint32_t M, uint32_t N, uint32_t K,
                            const GemmEpilogue& ep, uint32_t* err) {
   if (!A || !W || !M || !N || !K || (K & 7u) || (((uintptr_t)A | (uintptr_t)W) & 15)) return cudaErrorInvalidValue;
-  if ((ep.kind == GEMM_EPI_GATED || ep.kind == GEMM_EPI_QKV_ROPE) && (N & 1u)) return cudaErrorInvalidValue;
+  if ((ep.kind == GEMM_EPI_GATED || ep.kind == GEMM_EPI_GATED_CLAMPED || ep.kind == GEMM_EPI_QKV_ROPE) && (N & 1u)) return cudaErrorInvalidValue;
   if (ep.operands_bf16 > 1) return cudaErrorInvalidValue;
   // enough CTAs to pull weights with every SM when the chunk is a single row of tiles
   const uint32_t mtiles = (M + kBM - 1) / kBM;
@@ -720,7 +721,7 @@ cudaError_t launch_gemm_tc_grouped(cudaStream_t s, const __half* A, const __half
                                    const GemmGroups& g, const GemmEpilogue& ep, uint32_t* err) {
   static_assert(kGroupTile == kBM, "the tile list is made for this kernel's tiles");
   if (!A || !W || !max_rows || !N || !K || (K & 7u) || (((uintptr_t)A | (uintptr_t)W) & 15) || !g.count || !g.max_tiles) return cudaErrorInvalidValue;
-  if (ep.kind == GEMM_EPI_QKV_ROPE || (ep.kind == GEMM_EPI_GATED && (N & 1u)) || ep.bias || ep.resid || ep.operands_bf16 > 1) return cudaErrorInvalidValue;
+  if (ep.kind == GEMM_EPI_QKV_ROPE || ((ep.kind == GEMM_EPI_GATED || ep.kind == GEMM_EPI_GATED_CLAMPED) && (N & 1u)) || ep.bias || ep.resid || ep.operands_bf16 > 1) return cudaErrorInvalidValue;
   return launch_persistent<true>(s, A, W, max_rows, N, K, g, ep, err);
 }
 

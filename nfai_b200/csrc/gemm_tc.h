@@ -6,7 +6,7 @@
 
 namespace nfai {
 
-enum GemmEpilogueKind { GEMM_EPI_STORE = 0, GEMM_EPI_GATED = 1, GEMM_EPI_QKV_ROPE = 2, GEMM_EPI_STORE_ACT = 3 };
+enum GemmEpilogueKind { GEMM_EPI_STORE = 0, GEMM_EPI_GATED = 1, GEMM_EPI_QKV_ROPE = 2, GEMM_EPI_STORE_ACT = 3, GEMM_EPI_GATED_CLAMPED = 4 };
 
 struct GemmEpilogue {
   int kind = GEMM_EPI_STORE;
@@ -16,8 +16,9 @@ struct GemmEpilogue {
   void* out_act = nullptr;       // GATED: [M][N/2], STORE_ACT: [M][N], of out_dtype
   int out_dtype = 1;             // 0 float32, 1 float16, 2 bfloat16
   int act = 0;                   // GATED: Activation (kernels.h)
-  float act_limit = 0.f;         // GATED, clamped activation
-  uint32_t gated_cols = 0;       // GATED: only this many columns are gate/up pairs (0: all), the rest go plainly to out_f32
+  // GATED_CLAMPED: as GATED with the clamped activation and its limit, without bias
+  float act_limit = 0.f;
+  uint32_t gated_cols = 0;       // only this many columns are gate/up pairs (0: all), the rest go plainly to out_f32
                                  // [M][N - gated_cols]; even, as is N
   uint32_t operands_bf16 = 0;    // 1: A and W are bfloat16 (both), 0: float16 (both)
   // QKV_ROPE
@@ -52,8 +53,8 @@ uint32_t gemm_tc_splits(uint32_t M, uint32_t N, uint32_t K);
 cudaError_t launch_gemm_tc(cudaStream_t s, const __half* A, const __half* W, uint32_t M, uint32_t N, uint32_t K,
                            const GemmEpilogue& ep, uint32_t* err);
 
-// The same for grouped rows: A [rows][K] in group order, W [groups][N][K]; epilogues GATED, STORE and STORE_ACT without
-// bias or residual. max_rows bounds the rows of A.
+// The same for grouped rows: A [rows][K] in group order, W [groups][N][K]; epilogues GATED, GATED_CLAMPED, STORE and
+// STORE_ACT without bias or residual. max_rows bounds the rows of A.
 cudaError_t launch_gemm_tc_grouped(cudaStream_t s, const __half* A, const __half* W, uint32_t max_rows, uint32_t N, uint32_t K,
                                    const GemmGroups& g, const GemmEpilogue& ep, uint32_t* err);
 cudaError_t launch_gemm_simt_grouped(cudaStream_t s, int dtype, const void* A, const void* W, uint32_t N, uint32_t K, const GemmGroups& g,

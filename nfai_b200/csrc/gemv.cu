@@ -26,7 +26,9 @@ using namespace gemv_detail;
 // gemv_bf16.cu
 cudaError_t launch_gemv_more(int wdtype, GemvEpilogue epi, bool vec, int R, int U, dim3 grid, size_t smem, cudaStream_t s,
                              bool pdl, const GemvParams& p);
-// gemv_moe.cu
+// gemv_post.cu, gemv_moe.cu
+cudaError_t launch_gemv_post(int wdtype, GemvEpilogue epi, bool vec, int R, int U, dim3 grid, size_t smem, cudaStream_t s,
+                             bool pdl, const GemvParams& p);
 cudaError_t launch_gemv_experts(int wdtype, GemvEpilogue epi, bool vec, int R, int U, dim3 grid, size_t smem, cudaStream_t s,
                                 bool pdl, const GemvParams& p);
 
@@ -57,7 +59,7 @@ cudaError_t launch_e(GemvEpilogue epi, bool vec, int R, int U, dim3 grid, size_t
 
 bool vector_ok(int wdtype, const GemvParams& p) {
   const uint32_t ve = wdtype == 0 ? 4 : 8;
-  if (p.map == MAP_EXPERT_COLUMNS && (p.expert.seg % ve != 0 || (reinterpret_cast<uintptr_t>(p.expert.W2) & 15) != 0)) return false;
+  if (p.form == FORM_EXPERT_COLUMNS && (p.expert.seg % ve != 0 || (reinterpret_cast<uintptr_t>(p.expert.W2) & 15) != 0)) return false;
   return p.K % ve == 0 && (reinterpret_cast<uintptr_t>(p.W) & 15) == 0;
 }
 
@@ -72,7 +74,7 @@ int rows_per_warp(GemvEpilogue epi, bool vec, const GemvTune& t) {
 
 static bool use_ring(int wdtype, GemvEpilogue epi, const GemvParams& p, const GemvTune& t) {
   if (t.mode != 1 || !vector_ok(wdtype, p)) return false;
-  if (wdtype == 2 || epi == EPI_HYPER || p.norm_groups > 1 || p.y_ring || p.post.y || p.map || p.gated_rows) return false;
+  if (wdtype == 2 || epi == EPI_HYPER || p.norm_groups > 1 || p.y_ring || p.form) return false;
   return t.unroll >= 1 && t.unroll <= 4 && gemv_ring_smem(p, t.unroll) <= 227 * 1024;
 }
 
@@ -135,16 +137,19 @@ cudaError_t launch_gemv(cudaStream_t s, int wdtype, int kvdtype, GemvEpilogue ep
   dim3 grid(gemv_grid(wdtype, epi, p, t));
   p.split_log2 = gemv_split_log2(wdtype, vec, R, p, t);
   if (p.norm_groups > 1 && (!p.gain || p.K % p.norm_groups)) return cudaErrorInvalidValue;
+  if (p.form != FORM_POST_NORM && (p.post.y || p.gated_rows || p.gain_stride != 1)) return cudaErrorInvalidValue;
+  if (p.form == FORM_PLAIN && p.act == ACT_CLAMPED) return cudaErrorInvalidValue;
   if (p.gated_rows && (epi != EPI_GATED || !p.tail || (p.gated_rows & 1u))) return cudaErrorInvalidValue;
   if (p.post.y && (!p.post.gain || p.tp.pull || p.norm_groups > 1)) return cudaErrorInvalidValue;
-  size_t smem = (kSmemHeader + (size_t)gemv_x_floats(p) + gemv_map_floats(p, wdtype == 0 ? 4 : 8)) * sizeof(float);
+  size_t smem = (kSmemHeader + (size_t)gemv_x_floats(p) + gemv_form_floats(p, wdtype == 0 ? 4 : 8)) * sizeof(float);
   if (smem > 227 * 1024) return cudaErrorInvalidValue;
-  if (p.map) {
+  if (p.form == FORM_POST_NORM) return launch_gemv_post(wdtype, epi, vec, R, t.unroll, grid, smem, s, pdl, p);
+  if (p.form) {
     const ExpertMap& x = p.expert;
-    if (p.map == MAP_EXPERT_ROWS && (epi != EPI_GATED || !x.rows || (x.rows & 1u) || p.N != x.router.top * x.rows || !x.logits || !x.chosen ||
+    if (p.form == FORM_EXPERT_ROWS && (epi != EPI_GATED || !x.rows || (x.rows & 1u) || p.N != x.router.top * x.rows || !x.logits || !x.chosen ||
                                      x.router.top > 32 || x.router.experts > kMaxExperts || x.router.groups > kMaxGroups))
       return cudaErrorInvalidValue;
-    if (p.map == MAP_EXPERT_COLUMNS && (epi != EPI_STORE || !x.seg || !x.chosen || p.K < x.top * x.seg || (p.K > x.top * x.seg && (!x.W2 || !x.shared_gate))))
+    if (p.form == FORM_EXPERT_COLUMNS && (epi != EPI_STORE || !x.seg || !x.chosen || p.K < x.top * x.seg || (p.K > x.top * x.seg && (!x.W2 || !x.shared_gate))))
       return cudaErrorInvalidValue;
     return launch_gemv_experts(wdtype, epi, vec, R, t.unroll, grid, smem, s, pdl, p);
   }

@@ -11,10 +11,11 @@ constexpr int kWarps = kThreads / 32;
 
 // ---- prologue: x (optionally RMS-normalised) into shared memory ----------------------------------------------
 // The gain is a weight: it can be staged in shared memory before the programmatic-dependency wait.
+template <bool POST = false>
 __device__ __forceinline__ void load_gain(const GemvParams& p, float* xs, float* gs_at = nullptr) {
   if (p.gain == nullptr) return;
   float* gs = gs_at ? gs_at : xs + p.K;
-  for (uint32_t i = threadIdx.x; i < p.K; i += kThreads) gs[i] = p.gain[i * p.gain_stride];
+  for (uint32_t i = threadIdx.x; i < p.K; i += kThreads) gs[i] = p.gain[POST ? i * p.gain_stride : i];
 }
 
 // Tensor-parallel input: x = residual + the partial vectors of all ranks, which the previous row-parallel GEMV of
@@ -147,7 +148,7 @@ __device__ __forceinline__ float load_post_norm(const GemvParams& p, float* xs, 
 
 // ss = sum x^2 ; rms = sqrt(ss/K + eps) ; xs = (x / rms) * gain   (RMSNormShader.cs:136-148)
 // With PERM the shared-memory area of x must be a whole number of 256-element blocks.
-template <bool PERM = false>
+template <bool PERM = false, bool POST = false>
 __device__ __forceinline__ void load_x(const GemvParams& p, float* xs, float* red, const float* gs_in = nullptr) {
   const uint32_t K = p.K;
   const int tid = threadIdx.x;
@@ -157,8 +158,14 @@ __device__ __forceinline__ void load_x(const GemvParams& p, float* xs, float* re
   const float* gs = gs_in ? gs_in : xs + K;  // staged by load_gain() before the dependency wait
   const bool norm = p.gain != nullptr;
   float ss = 0.f;
-  if (!PERM && p.post.y) {
-    ss = load_post_norm(p, xs, xs + (norm ? 2 : 1) * K, red);
+  bool loaded = false;
+  if constexpr (POST) {
+    if (p.post.y) {
+      ss = load_post_norm(p, xs, xs + (norm ? 2 : 1) * K, red);
+      loaded = true;
+    }
+  }
+  if (POST && loaded) {
   } else if (pull) {  // the host guarantees K % 4 == 0 and 16-byte aligned vectors for a pulling kernel
     const uint32_t pull_epoch = *p.tp.epoch_base + p.tp.pull_index + 1;
     bool pull_ok = true;
@@ -327,12 +334,7 @@ __device__ __forceinline__ void row_epilogue(const GemvParams& p, uint32_t row0,
       if (n >= p.N) break;
       // sigmoid = 1/(1+exp(-x)); silu = x*sigmoid; h = up*silu (SiLUShader.cs:121-123, ElementWiseMul A=up,B=silu)
       const float gate = p.bias ? acc[r] + __ldg(p.bias + n) : acc[r], up = p.bias ? acc[r + 1] + __ldg(p.bias + n + 1) : acc[r + 1];
-      if (p.gated_rows && n >= p.gated_rows) {  // (n is even, and so is gated_rows)
-        p.tail[n - p.gated_rows] = acc[r];
-        if (n + 1 < p.N) p.tail[n + 1 - p.gated_rows] = acc[r + 1];
-        continue;
-      }
-      p.y[n >> 1] = gated(p.act, gate, up, p.act_limit);
+      p.y[n >> 1] = gated(p.act, gate, up);
     }
   } else {  // EPI_LOGITS: store and keep the warp's best (lowest index among equal maxima)
 #pragma unroll
@@ -388,7 +390,10 @@ __device__ __forceinline__ void epi_preload(const GemvParams& p, uint32_t row0, 
   }
 }
 
-template <typename KVT, int R, int EPI, int MAP = MAP_PLAIN>
+__device__ __forceinline__ float any_gated(const GemvParams& p, float gate, float up) {
+  return p.act == ACT_CLAMPED ? gated_clamped(gate, up, p.act_limit) : gated(p.act, gate, up);
+}
+template <typename KVT, int R, int EPI, int FORM = FORM_PLAIN>
 __device__ __forceinline__ void row_epilogue_pre(const GemvParams& p, uint32_t row0, const float (&acc)[R],
                                                  const float (&pre)[R], uint32_t pos, float& best_v, uint32_t& best_i) {
   if constexpr (EPI == EPI_HYPER) {  // the whole warp: lane t makes stream t
@@ -417,11 +422,26 @@ __device__ __forceinline__ void row_epilogue_pre(const GemvParams& p, uint32_t r
     return;
   }
   if ((threadIdx.x & 31) != 0) return;
-  if constexpr (MAP == MAP_EXPERT_ROWS) {  // `pre` holds the weights of the rows' experts
+  if constexpr (FORM == FORM_EXPERT_ROWS) {  // `pre` holds the weights of the rows' experts
     static_assert(EPI == EPI_GATED && R % 2 == 0, "gate and up rows are interleaved");
 #pragma unroll
     for (int r = 0; r < R; r += 2)
-      if (row0 + r < p.N) p.y[(row0 + r) >> 1] = pre[r] * gated(p.act, acc[r], acc[r + 1], p.act_limit);
+      if (row0 + r < p.N) p.y[(row0 + r) >> 1] = pre[r] * any_gated(p, acc[r], acc[r + 1]);
+    return;
+  }
+  if constexpr (FORM == FORM_POST_NORM && EPI == EPI_GATED) {
+#pragma unroll
+    for (int r = 0; r < R; r += 2) {
+      const uint32_t n = row0 + r;  // (even, as is gated_rows)
+      if (n >= p.N) break;
+      const float a = p.bias ? acc[r] + __ldg(p.bias + n) : acc[r], b = p.bias ? acc[r + 1] + __ldg(p.bias + n + 1) : acc[r + 1];
+      if (p.gated_rows && n >= p.gated_rows) {
+        p.tail[n - p.gated_rows] = a;
+        if (n + 1 < p.N) p.tail[n + 1 - p.gated_rows] = b;
+      } else {
+        p.y[n >> 1] = any_gated(p, a, b);
+      }
+    }
     return;
   }
   if constexpr (EPI == EPI_STORE) {

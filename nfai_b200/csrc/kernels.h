@@ -86,7 +86,7 @@ constexpr uint32_t kPrefetchChunk = 4096;
 enum GemvEpilogue {
   EPI_STORE = 0,     // y = acc (+ resid)
   EPI_QKV_ROPE = 1,  // rows are [Q | K | V]; RoPE on Q and K; K,V rows go to the cache at row pos
-  EPI_GATED = 2,     // rows are interleaved (gate_j, up_j); h_j = up_j * act(gate_j); rows from gated_rows on are stored plainly
+  EPI_GATED = 2,     // rows are interleaved (gate_j, up_j); h_j = up_j * act(gate_j)
   EPI_LOGITS = 3,    // y = acc and a per-CTA (max, lowest index) partial
   EPI_HYPER = 4      // y = acc is written into all residual streams (hyper-connections, see HyperWrite)
 };
@@ -124,18 +124,21 @@ struct Router {
   float scale = 1.f;
 };
 
-// How a GEMV finds its weights when the chosen experts decide.
-//   MAP_EXPERT_ROWS    W is [experts][rows][K]; row n of the product is row n % rows of the (n / rows)-th chosen expert, its
+// What a GEMV kernel is compiled for; the plain form carries none of the others' code.
+//   FORM_POST_NORM   plain weights; the prologue knows PostNorm and gains of one number, the gated epilogue the clamped
+//                    activation and plain rows behind the gated ones.
+// The others find their weights through the chosen experts, and know the clamped activation:
+//   FORM_EXPERT_ROWS    W is [experts][rows][K]; row n of the product is row n % rows of the (n / rows)-th chosen expert, its
 //                      gated output times that expert's weight. Every CTA works the choice out for itself; CTA 0 keeps it.
-//   MAP_EXPERT_COLUMNS the product over K = [top x seg | shared]: part k of x meets row n of W + chosen[k] * N * seg, the last
+//   FORM_EXPERT_COLUMNS the product over K = [top x seg | shared]: part k of x meets row n of W + chosen[k] * N * seg, the last
 //                      part meets W2 and is first multiplied by the sigmoid of *shared_gate.
-enum WeightMap { MAP_PLAIN = 0, MAP_EXPERT_ROWS = 1, MAP_EXPERT_COLUMNS = 2 };
+enum GemvForm { FORM_PLAIN = 0, FORM_EXPERT_ROWS = 1, FORM_EXPERT_COLUMNS = 2, FORM_POST_NORM = 3 };
 struct ExpertMap {
   Router router;
-  const float* logits = nullptr;  // MAP_EXPERT_ROWS
-  uint32_t rows = 0;              // MAP_EXPERT_ROWS: rows per expert (even)
+  const float* logits = nullptr;  // FORM_EXPERT_ROWS
+  uint32_t rows = 0;              // FORM_EXPERT_ROWS: rows per expert (even)
   uint32_t* chosen = nullptr;     // [top], written / read
-  uint32_t seg = 0, top = 0;      // MAP_EXPERT_COLUMNS
+  uint32_t seg = 0, top = 0;      // FORM_EXPERT_COLUMNS
   const void* W2 = nullptr;       // [N][K - top*seg]
   const float* shared_gate = nullptr;
 };
@@ -176,12 +179,13 @@ struct GemvParams {
   // EPI_STORE into a ring of rows: y is row (position % y_ring) of a buffer of rows y_stride floats apart (0 = plain y)
   uint32_t y_ring = 0, y_stride = 0;
   HyperWrite hyper;             // EPI_HYPER
-  float act_limit = 0.f;        // EPI_GATED, clamped activation
+  int form = FORM_PLAIN;
+  float act_limit = 0.f;        // clamped activation (not FORM_PLAIN)
+  // FORM_POST_NORM
   uint32_t gain_stride = 1;     // 0: gain is one number for all of x
   PostNorm post;
   uint32_t gated_rows = 0;      // EPI_GATED: rows from here on are stored plainly to tail (even; 0: none)
   float* tail = nullptr;
-  int map = MAP_PLAIN;
   ExpertMap expert;
 };
 

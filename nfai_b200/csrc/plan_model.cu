@@ -178,6 +178,8 @@ static int plan_create(nfai_ctx* c, LayerPlan&& plan_in, uint32_t ctx_size, int 
     std::string why;
     if (l.mixer == MIXER_LATENT && !latent_supported(l.latent, weight_dtype, &why)) return fail(c, NFAI_ERR_ARG, "%s", why.c_str());
     if (l.mixer == MIXER_GQA && !gqa_supported(l.gqa, &why)) return fail(c, NFAI_ERR_ARG, "%s", why.c_str());
+    if (l.mlp == FF_MOE && (pl.act != ACT_CLAMPED || pl.residual != RESIDUAL_POST_NORM))
+      return fail(c, NFAI_ERR_ARG, "routed feed-forwards come with the clamped activation and a post-norm residual");
   }
   P->act_dtype = weight_dtype;
   nfai_hparams& hp = m->hp;
@@ -602,6 +604,7 @@ bool post_norm(const nfai_model* m) { return m->plan->plan.residual == RESIDUAL_
 // and what to add to it; it keeps the sum.
 void behind(nfai_model* m, GemvParams& p, uint32_t layer, int q, uint32_t sub) {
   PlanModel* P = m->plan.get();
+  p.form = FORM_POST_NORM;
   p.x = streams(m, sub);
   p.post.y = P->y;
   p.post.gain = P->w[layer].sub[q].norm.ptr;
@@ -619,6 +622,7 @@ void reader(nfai_model* m, GemvParams& p, uint32_t l, int q, uint32_t sub) {
     p.gain = P->w[l].sub[q].norm.ptr;
     p.eps = m->hp.eps;
   } else if (sub == 0) {
+    p.form = FORM_POST_NORM;
     p.x = streams(m, 0);
   } else {
     if (q) behind(m, p, l, 0, sub - 1);
@@ -744,7 +748,7 @@ GemvParams expert_params(nfai_model* m, uint32_t l, uint32_t sub) {
   p.act = P->plan.act;
   p.act_limit = s.limit;
   p.y = P->hbuf;
-  p.map = MAP_EXPERT_ROWS;
+  p.form = FORM_EXPERT_ROWS;
   p.expert.router = router_of(m, l);
   p.expert.logits = P->tail;
   p.expert.rows = 2 * s.ff;
@@ -759,7 +763,7 @@ GemvParams expert_down_params(nfai_model* m, uint32_t l, uint32_t sub) {
   p.W = P->w[l].exp_down.ptr;
   p.K = s.hidden();
   p.x = P->hbuf;
-  p.map = MAP_EXPERT_COLUMNS;
+  p.form = FORM_EXPERT_COLUMNS;
   p.expert.chosen = P->chosen;
   p.expert.seg = s.ff;
   p.expert.top = s.top;
@@ -848,6 +852,7 @@ GemvParams plan_head_params(nfai_model* m, bool settled) {
   p.x = m->plan->u;
   if (post_norm(m)) {
     const uint32_t last = pl.sublayers();
+    p.form = FORM_POST_NORM;
     if (settled) p.x = streams(m, last);
     else behind(m, p, m->hp.L - 1, pl.layers.back().has_mlp() ? 1 : 0, last - 1);
   }
@@ -1010,8 +1015,7 @@ cudaError_t moe_pass(nfai_model* m, uint32_t l, uint32_t T) {
   const uint32_t H = m->hp.H;
   cudaError_t e;
   GemmEpilogue ef;
-  ef.kind = sp.shared_ff ? GEMM_EPI_GATED : GEMM_EPI_STORE;
-  ef.act = P->plan.act;
+  ef.kind = sp.shared_ff ? GEMM_EPI_GATED_CLAMPED : GEMM_EPI_STORE;
   ef.act_limit = sp.shared_limit;
   ef.gated_cols = sp.gated_rows();
   ef.out_act = P->pF;
@@ -1031,8 +1035,7 @@ cudaError_t moe_pass(nfai_model* m, uint32_t l, uint32_t T) {
   g.n_tiles = r.n_tiles;
   g.max_tiles = moe_max_tiles(sp, T);
   GemmEpilogue eg;
-  eg.kind = GEMM_EPI_GATED;
-  eg.act = P->plan.act;
+  eg.kind = GEMM_EPI_GATED_CLAMPED;
   eg.act_limit = sp.limit;
   eg.out_act = P->pFE;
   if ((e = grouped_product(m, P->pG, w.exp_gateup.ptr, pairs, 2 * sp.ff, H, g, eg)) != cudaSuccess) return e;
@@ -1052,7 +1055,7 @@ cudaError_t mlp_pass(nfai_model* m, uint32_t l, uint32_t T) {
   const uint32_t H = m->hp.H;
   if (pl.mlp == FF_MOE) return moe_pass(m, l, T);
   GemmEpilogue eg;
-  eg.kind = GEMM_EPI_GATED;
+  eg.kind = P->plan.act == ACT_CLAMPED ? GEMM_EPI_GATED_CLAMPED : GEMM_EPI_GATED;
   eg.act = P->plan.act;
   eg.act_limit = pl.limit;
   eg.bias = w.gateup_b.ptr;
